@@ -3,11 +3,11 @@ and slots for fixed-size per-request state.
 
 Each call of the model's schedule that owns a cache declares what it needs
 (:class:`PagedKVNeed`, :class:`StateNeed` or nothing).  Calls with the same page shape and
-the same window form a *group*: one pool of pages, one block table per request.  A page id
+the same window (or chunk size) form a *group*: one pool of pages, one block table per request.  A page id
 means the same page in every call of its group, so a request's table is one row per group
 however many layers there are (the reference keeps one table per layer,
 include/backend/kvcache/block_pool.hpp:73-103).  Groups with a window give pages back as soon
-as the window has passed them; everything is given back when a request is closed.
+as the window has passed them, groups with chunks when the next token opens a new chunk; everything is given back when a request is closed.
 
 Device layout of a group: ``[num_pages + 1, calls, planes, kv_heads, page_size, head_dim]``; the usual cache has two
 planes (keys, values), a cache whose rows are keys and values at once (the latent of a latent-attention layer) has one.
@@ -31,6 +31,7 @@ class PagedKVNeed:
     head_dim: int
     window: Optional[int] = None        # None: all keys; else the last `window` keys
     planes: int = 2                     # 2: keys and values; 1: one row per token that serves as both (a latent)
+    chunk: Optional[int] = None         # keys of the query's own chunk of that many positions alone (chunks counted from 0)
 
 
 @dataclass(frozen=True)
@@ -57,10 +58,24 @@ class PagedGroup:
     head_dim: int
     window: Optional[int]
     planes: int = 2
+    chunk: Optional[int] = None
     calls: List[int] = field(default_factory=list)
     pool: Optional[PagePool] = None
     tensor: Optional[torch.Tensor] = None
     num_pages: int = 0                  # pages of this group's pool; page ``num_pages`` of the tensor is the scratch page
+
+    @property
+    def span(self) -> Optional[int]:
+        """The most keys a query may see, where that is bounded (a window or a chunk); None: every key."""
+        return self.window if self.window is not None else self.chunk
+
+    def first_needed_token(self, length: int) -> int:
+        """The first token that a request of ``length`` committed tokens still needs: its next query sits at ``length``."""
+        if self.window is not None:
+            return max(0, length - self.window + 1)
+        if self.chunk is not None:
+            return length // self.chunk * self.chunk
+        return 0
 
     def page_elems(self, page_size: int) -> int:
         return len(self.calls) * self.planes * self.n_kv_heads * page_size * self.head_dim
@@ -105,13 +120,16 @@ class CacheManager:
                 continue
             if isinstance(need, PagedKVNeed):
                 for gi, g in enumerate(self.groups):
-                    if (g.n_kv_heads, g.head_dim, g.window, g.planes) == (need.n_kv_heads, need.head_dim, need.window, need.planes):
+                    if (g.n_kv_heads, g.head_dim, g.window, g.planes, g.chunk) == (need.n_kv_heads, need.head_dim, need.window, need.planes,
+                                                                                      need.chunk):
                         break
                 else:
                     if need.planes not in (1, 2):
                         raise ValueError(f"call {call}: a paged cache has 1 or 2 planes, not {need.planes}")
                     gi = len(self.groups)
-                    self.groups.append(PagedGroup(need.n_kv_heads, need.head_dim, need.window, need.planes))
+                    if need.window is not None and need.chunk is not None:
+                        raise ValueError(f"call {call}: a paged cache keeps a window or chunks, not both")
+                    self.groups.append(PagedGroup(need.n_kv_heads, need.head_dim, need.window, need.planes, need.chunk))
                 self._call_group[call] = (gi, len(self.groups[gi].calls))
                 self.groups[gi].calls.append(call)
             elif isinstance(need, StateNeed):
@@ -140,11 +158,11 @@ class CacheManager:
 
     def group_pages(self, g: PagedGroup, num_pages: int) -> int:
         """Pages of group ``g`` when the groups that keep all keys get ``num_pages``: as many, or, for a group with a
-        window under a bound on a step's tokens, what ``max_requests`` requests can hold at most."""
-        if g.window is None or self.max_step_tokens is None:
+        window or chunks under a bound on a step's tokens, what ``max_requests`` requests can hold at most."""
+        if g.span is None or self.max_step_tokens is None:
             return num_pages
-        # window - 1 + step tokens, starting anywhere in a page
-        per_request = (g.window + self.max_step_tokens + self.page_size - 2) // self.page_size + 1
+        # span - 1 + step tokens, starting anywhere in a page
+        per_request = (g.span + self.max_step_tokens + self.page_size - 2) // self.page_size + 1
         return max(1, min(num_pages, per_request * self.max_requests))
 
     def pool_bytes(self, num_pages: int, dtype: torch.dtype) -> int:
@@ -194,7 +212,7 @@ class CacheManager:
     def step_bound(self) -> Optional[int]:
         """The most tokens of one request that a step may bring, where the pools rely on it (some group has a window
         and the caller gave ``max_step_tokens``); None where nothing depends on it."""
-        if self.max_step_tokens is not None and any(g.window is not None for g in self.groups):
+        if self.max_step_tokens is not None and any(g.span is not None for g in self.groups):
             return self.max_step_tokens
         return None
 
@@ -266,10 +284,7 @@ class CacheManager:
 
     def _first_needed_block(self, g: PagedGroup, length: int) -> int:
         """Index of the first block a request of ``length`` committed tokens still needs."""
-        if g.window is None:
-            return 0
-        first_token = max(0, length - g.window + 1)      # the next query (position >= length) reads from here
-        return first_token // self.page_size
+        return g.first_needed_token(length) // self.page_size
 
     def pages_needed(self, rc: Optional[RequestCache], new_len: int) -> List[int]:
         """Pages per group that ``ensure(rc, new_len)`` would take (``rc=None``: a fresh request).  A group with a
@@ -280,7 +295,7 @@ class CacheManager:
         out = []
         for gi, g in enumerate(self.groups):
             reach = new_len
-            if g.window is not None and self.max_step_tokens is not None:
+            if g.span is not None and self.max_step_tokens is not None:
                 reach = min(new_len, length + self.max_step_tokens)
             want = (reach + self.page_size - 1) // self.page_size
             have = len(rc.tables[gi]) if rc is not None else 0
@@ -312,7 +327,7 @@ class CacheManager:
             raise ValueError("a request's length cannot shrink")
         rc.length = new_len
         for gi, g in enumerate(self.groups):
-            if g.window is None:
+            if g.span is None:
                 continue
             table = rc.tables[gi]
             for b in range(min(self._first_needed_block(g, new_len), len(table))):

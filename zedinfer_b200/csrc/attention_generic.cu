@@ -3,8 +3,8 @@
 // heads and groups, any page size, and an optional window.
 //
 // This kernel is the whole 32-bit path and the general fallback of the bfloat16 path.  A query
-// at absolute position P sees the keys lo..P of its own request, lo = max(0, P - window + 1)
-// (window 0 = all keys).  Keys are visited in tiles of 32 starting at lo with one online-softmax
+// at absolute position P sees the keys lo..P of its own request, lo = first_visible_key(P, window)
+// (window 0 = all keys, > 0 the last ones, < 0 those of its own chunk).  Keys are visited in tiles of 32 starting at lo with one online-softmax
 // rule, so the result for a query depends on P and the cache contents alone: not on how the
 // prompt was cut into steps, nor on what else is in the batch.
 //
@@ -16,6 +16,7 @@
 // key and no value; it is added once, after the last tile, relative to the running maximum of the scores.
 //
 // softcap c > 0: a score s (after the scale) becomes c * tanh(s / c) before the softmax.
+// bias: a number per query head and distance P - j that is added to the score after that.
 #include "zi_common.cuh"
 
 ZI_DEFINE_LAST_ERROR(attention_generic)
@@ -29,7 +30,7 @@ paged_attention_kernel(const T* __restrict__ q, const T* __restrict__ cache, T* 
                        const int* __restrict__ tables, const int* __restrict__ tok_seg,
                        const int* __restrict__ pos, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                        int page_size, int max_blocks, long long page_stride, long long kv_stride, int window,
-                       float scale, const float* __restrict__ sinks, float softcap) {
+                       float scale, const float* __restrict__ sinks, float softcap, const DistanceBias bias) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* qs = smem + warp * head_dim;                                     // this warp's query
@@ -39,7 +40,8 @@ paged_attention_kernel(const T* __restrict__ q, const T* __restrict__ cache, T* 
     const int n = (int)(item / n_heads), h = (int)(item - (long long)n * n_heads);
     const int kvh = h / (n_heads / n_kv_heads);
     const int P = pos[n];
-    const int lo = (window > 0 && P - window + 1 > 0) ? P - window + 1 : 0;
+    const int lo = first_visible_key(P, window);
+    const float* bias_row = bias.table ? bias.table + (size_t)h * bias.len : nullptr;
     const int* table = tables + (size_t)tok_seg[n] * max_blocks;
     const T* qrow = q + ((size_t)n * n_heads + h) * head_dim;
     for (int d = lane; d < head_dim; d += 32) qs[d] = to_f32<T>(qrow[d]);
@@ -68,6 +70,7 @@ paged_attention_kernel(const T* __restrict__ q, const T* __restrict__ cache, T* 
             }
             s = dot * scale;
             if (softcap > 0.0f) s = softcap * tanhf(s / softcap);
+            if (bias_row) s += bias_row[min(P - j, bias.len - 1)];
         }
         rows[lane] = roff;
         const float m_new = fmaxf(m, warp_max(s));
@@ -104,13 +107,14 @@ ZI_EXPORT int zi_paged_attention(const void* q, const void* cache, void* out, in
                                  const int* tok_seg, const int* pos, int n_tokens, int n_heads, int n_kv_heads,
                                  int head_dim, int page_size, int max_blocks, long long page_stride,
                                  long long kv_stride, int window, float scale, const float* sinks, float softcap,
-                                 cudaStream_t stream) {
+                                 const float* bias, int bias_len, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (head_dim <= 0 || head_dim % 8 != 0 || head_dim > 1024)
         return zi_fail("attention: head_dim=%d must be a multiple of 8 and at most %d", head_dim, 1024);
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0)
         return zi_fail("attention: %d query heads cannot share %d key/value heads", n_heads, n_kv_heads);
     if (page_size <= 0 || max_blocks <= 0) return zi_fail("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
+    if (bias && bias_len <= 0) return zi_fail("attention: a table of %d distances", bias_len);
     const long long items = (long long)n_tokens * n_heads;
     const long long blocks = (items + WARPS - 1) / WARPS;
     if (blocks > 0x7fffffffLL) return zi_fail("attention: too many (token, head) pairs: %lld", items);
@@ -119,15 +123,15 @@ ZI_EXPORT int zi_paged_attention(const void* q, const void* cache, void* out, in
         if (head_dim <= 256)
             paged_attention_kernel<T, 8><<<(unsigned)blocks, WARPS * 32, smem, stream>>>(
                 (const T*)q, (const T*)cache, (T*)out, tables, tok_seg, pos, n_tokens, n_heads, n_kv_heads, head_dim,
-                page_size, max_blocks, page_stride, kv_stride, window, scale, sinks, softcap);
+                page_size, max_blocks, page_stride, kv_stride, window, scale, sinks, softcap, DistanceBias{bias, bias_len});
         else if (head_dim <= 512)
             paged_attention_kernel<T, 16><<<(unsigned)blocks, WARPS * 32, smem, stream>>>(
                 (const T*)q, (const T*)cache, (T*)out, tables, tok_seg, pos, n_tokens, n_heads, n_kv_heads, head_dim,
-                page_size, max_blocks, page_stride, kv_stride, window, scale, sinks, softcap);
+                page_size, max_blocks, page_stride, kv_stride, window, scale, sinks, softcap, DistanceBias{bias, bias_len});
         else
             paged_attention_kernel<T, 32><<<(unsigned)blocks, WARPS * 32, smem, stream>>>(
                 (const T*)q, (const T*)cache, (T*)out, tables, tok_seg, pos, n_tokens, n_heads, n_kv_heads, head_dim,
-                page_size, max_blocks, page_stride, kv_stride, window, scale, sinks, softcap);
+                page_size, max_blocks, page_stride, kv_stride, window, scale, sinks, softcap, DistanceBias{bias, bias_len});
     });
     return zi_check_launch("paged_attention");
 }

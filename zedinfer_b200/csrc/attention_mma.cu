@@ -1,5 +1,5 @@
 // Paged causal attention for bfloat16 on the tensor cores (mma.sync m16n8k16, float32 accumulate),
-// head_dim 64 or 128, any number of heads and groups, any page size, optional window.
+// head_dim 64 or 128, any number of heads and groups, any page size, optional window or chunks, optional bias by distance.
 //
 //   decode  : one query token per request.  The query heads that share a key/value head form the
 //             rows of one 16-row tile, so the keys and values of a request cross the memory bus once
@@ -162,6 +162,30 @@ __device__ __forceinline__ void cap_scores(float (&S)[NKT][4], float cap_in) {
     }
 }
 
+// Bias by distance on a warp's score tile.  Rows g and g + 8 of the tile have the table rows t0 and t1 and, at the tile's first
+// key, the distances d0 and d1; the scores are raw dot products, so the table's numbers come in divided by what multiplies a
+// raw score (inv).  A tile farther away than the table reaches gets each row's last entry.
+template <int NKT>
+__device__ __forceinline__ void bias_scores(float (&S)[NKT][4], const float* __restrict__ t0, const float* __restrict__ t1, int d0, int d1,
+                                            int last, float inv, int lane) {
+    if (min(d0, d1) - (NKT * 8 - 1) >= last) {
+        const float b0 = __ldg(t0 + last) * inv, b1 = __ldg(t1 + last) * inv;
+#pragma unroll
+        for (int nt = 0; nt < NKT; ++nt) { S[nt][0] += b0; S[nt][1] += b0; S[nt][2] += b1; S[nt][3] += b1; }
+        return;
+    }
+    const int at = (lane & 3) * 2;
+#pragma unroll
+    for (int nt = 0; nt < NKT; ++nt) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int off = nt * 8 + at + e;
+            S[nt][e] = fmaf(__ldg(t0 + min(max(d0 - off, 0), last)), inv, S[nt][e]);          // distances below 0 are masked afterwards
+            S[nt][2 + e] = fmaf(__ldg(t1 + min(max(d1 - off, 0), last)), inv, S[nt][2 + e]);
+        }
+    }
+}
+
 // Online softmax step on a warp's score tile.  Thread holds rows g = lane/4 (values [0],[1]) and g+8
 // ([2],[3]) at keys key0 + nt*8 + (lane%4)*2 + {0,1}.  lo / hi: first / last key each row may see.
 // S comes in as raw dot products and leaves as probabilities relative to the running maximum; m is kept
@@ -230,7 +254,7 @@ decode_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cac
                         const int* __restrict__ tables, const int* __restrict__ tok_seg,
                         const int* __restrict__ pos, int n_heads, int n_kv_heads, int q_blocks, int page_size,
                         int page_shift, int max_blocks, long long page_stride, long long kv_stride, int window,
-                        float scale2, const float* __restrict__ sinks, float cap_in) {
+                        float scale2, const float* __restrict__ sinks, float cap_in, const DistanceBias bias, float bias_inv) {
     namespace cg = cooperative_groups;
     cg::cluster_group cluster = cg::this_cluster();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -244,7 +268,7 @@ decode_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cac
     pdl_trigger_early();
     pdl_wait();
     const int P = ld_dep(pos + n);
-    const int lo = (window > 0 && P - window + 1 > 0) ? P - window + 1 : 0;
+    const int lo = first_visible_key(P, window);
     const int t_lo = lo / TILE_KEYS, t_hi = P / TILE_KEYS;
     const int n_mine = (t_hi - t_lo - rank >= 0) ? (t_hi - t_lo - rank) / DEC_CLUSTER + 1 : 0;
 
@@ -271,6 +295,9 @@ decode_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cac
         }
         *reinterpret_cast<uint4*>(smem_raw + swz<HD>(row, c)) = v;
     }
+    const int bias_h0 = kvh * group + qb * 16;                    // rows past the group's heads take its first head's entries
+    const float* bias0 = bias.table + (size_t)(bias_h0 + ((lane >> 2) < rows_valid ? (lane >> 2) : 0)) * bias.len;
+    const float* bias1 = bias.table + (size_t)(bias_h0 + ((lane >> 2) + 8 < rows_valid ? (lane >> 2) + 8 : 0)) * bias.len;
     // prologue: the first DEC_STAGES tiles of this block; one commit group per stage whether it holds a tile or not
 #pragma unroll
     for (int s = 0; s < DEC_STAGES; ++s) {
@@ -302,6 +329,7 @@ decode_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cac
             float S[2][4];
             qk_scores<HD, 2>(S, qf, sK, warp * 16, lane);
             cap_scores<2>(S, cap_in);
+            if (bias.table) bias_scores<2>(S, bias0, bias1, P - key0, P - key0, bias.len - 1, bias_inv, lane);
             softmax_step<HD, 2>(S, O, m, l, key0, lane, lo, P, lo, P, scale2);
             pv_accumulate<HD, 2>(O, S, sV, warp * 16, lane);
         }
@@ -462,7 +490,7 @@ decode_attention_merge_kernel(const float* __restrict__ part, bf16* __restrict__
                               const float* __restrict__ sinks) {
     const int n = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
     const int P = pos[n];
-    const int lo = (window > 0 && P - window + 1 > 0) ? P - window + 1 : 0;
+    const int lo = first_visible_key(P, window);
     const int eff = dt_effective_splits(P / dt_keys - lo / dt_keys + 1, n_splits, min_split_tiles);
     if (eff == 1) return;
     const float* src = part + ((size_t)n * n_heads + h) * n_splits * (HD + 2);
@@ -485,7 +513,7 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const bf
                             int* __restrict__ status, int n_heads, int n_kv_heads, int q_blocks, int page_size,
                             int box_rows, int max_blocks, int window, float scale2, int n_splits, int min_split_tiles,
                             float* __restrict__ part, int kv_box, const float* __restrict__ sinks, int one_plane,
-                            float cap_in) {
+                            float cap_in, const DistanceBias bias, float bias_inv) {
     namespace cg = cooperative_groups;
     cg::cluster_group cluster = cg::this_cluster();
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -513,7 +541,7 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const bf
         if (blk < max_blocks) id_reg = table[blk];
     }
     const int P = pos[n];
-    const int lo = (window > 0 && P - window + 1 > 0) ? P - window + 1 : 0;
+    const int lo = first_visible_key(P, window);
     // The visible tiles may be shared out over several clusters (long contexts of few requests, see dt_splits): as
     // many of the n_splits as leave each at least min_split_tiles tiles.  Clusters beyond that number have nothing
     // to do; with more than one at work each leaves (m, l, O) in `part` and decode_attention_merge_kernel adds them.
@@ -609,6 +637,9 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const bf
     for (int dn = 0; dn < HD / 8; ++dn) O[dn][0] = O[dn][1] = O[dn][2] = O[dn][3] = 0.0f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 
+    const int bias_h0 = kvh * group + qb * 16;                    // rows past the group's heads take its first head's entries
+    const float* bias0 = bias.table + (size_t)(bias_h0 + ((lane >> 2) < rows_valid ? (lane >> 2) : 0)) * bias.len;
+    const float* bias1 = bias.table + (size_t)(bias_h0 + ((lane >> 2) + 8 < rows_valid ? (lane >> 2) + 8 : 0)) * bias.len;
     bool ok = true;
     int failed_at = 0;
     for (int i = 0; i < n_mine; ++i) {
@@ -619,6 +650,7 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const bf
         float S[DT_KEYS / 8][4];
         qk_scores_tma<HD, DT_KEYS / 8>(S, qf, sK, lane);
         cap_scores<DT_KEYS / 8>(S, cap_in);
+        if (bias.table) bias_scores<DT_KEYS / 8>(S, bias0, bias1, P - key0, P - key0, bias.len - 1, bias_inv, lane);
         if (key0 >= lo && key0 + DT_KEYS - 1 <= P) softmax_step<HD, DT_KEYS / 8, false>(S, O, m, l, key0, lane, lo, P, lo, P, scale2);
         else softmax_step<HD, DT_KEYS / 8, true>(S, O, m, l, key0, lane, lo, P, lo, P, scale2);
         pv_accumulate_tma<HD, DT_KEYS / 8>(O, S, sV, lane);
@@ -725,7 +757,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ ca
                          const int* __restrict__ tables, const int* __restrict__ tiles, const int* __restrict__ pos,
                          int n_heads, int n_kv_heads, int page_size, int page_shift, int max_blocks,
                          long long page_stride, long long kv_stride, int window, float scale2,
-                         const float* __restrict__ sinks, float cap_in) {
+                         const float* __restrict__ sinks, float cap_in, const DistanceBias bias, float bias_inv) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     constexpr int TILE_BYTES = TILE_KEYS * HD * 2;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -740,7 +772,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ ca
     const int kvh = h / (n_heads / n_kv_heads);
     const int p0 = pos[n0];                                       // positions of a portion are consecutive
     const int p_last = p0 + rows - 1;
-    const int lo_tile = (window > 0 && p0 - window + 1 > 0) ? p0 - window + 1 : 0;
+    const int lo_tile = first_visible_key(p0, window);
 
     CacheRef cr;
     cr.base = cache; cr.table = tables + (size_t)seg * max_blocks;
@@ -773,12 +805,12 @@ prefill_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ ca
     const int g = lane >> 2;
     const int r0 = warp * 16 + g, r1 = r0 + 8;
     const int hi0 = r0 < rows ? p0 + r0 : -1, hi1 = r1 < rows ? p0 + r1 : -1;      // padding rows see nothing
-    const int lo0 = (window > 0 && hi0 - window + 1 > 0) ? hi0 - window + 1 : 0;
-    const int lo1 = (window > 0 && hi1 - window + 1 > 0) ? hi1 - window + 1 : 0;
+    const int lo0 = first_visible_key(hi0, window);
+    const int lo1 = first_visible_key(hi1, window);
     // what this warp's 16 rows may see at most
     const int w_rows = rows - warp * 16;                         // rows of this warp that exist
     const int w_hi = p0 + warp * 16 + (w_rows < 16 ? w_rows : 16) - 1;
-    const int w_lo = (window > 0 && p0 + warp * 16 - window + 1 > 0) ? p0 + warp * 16 - window + 1 : 0;
+    const int w_lo = first_visible_key(p0 + warp * 16, window), w_hi_lo = first_visible_key(w_hi, window);
 
     for (int t = t_first; t <= t_last; ++t) {
         const int stage = (t - t_first) & 1;
@@ -797,9 +829,13 @@ prefill_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ ca
             float S[8][4];
             qk_scores<HD, 8>(S, qf, sK, 0, lane);
             cap_scores<8>(S, cap_in);
+            if (bias.table) {
+                const float* bt = bias.table + (size_t)h * bias.len;
+                bias_scores<8>(S, bt, bt, p0 + r0 - key0, p0 + r1 - key0, bias.len - 1, bias_inv, lane);
+            }
             // every existing row of the warp sees the whole tile: rows sit at p0 + warp*16 .. w_hi
             const bool full = w_rows >= 16 && key0 + TILE_KEYS - 1 <= p0 + warp * 16 &&
-                              (window <= 0 || key0 >= w_hi - window + 1);
+                              key0 >= w_hi_lo;
             if (full) softmax_step<HD, 8, false>(S, O, m, l, key0, lane, lo0, hi0, lo1, hi1, scale2);
             else softmax_step<HD, 8, true>(S, O, m, l, key0, lane, lo0, hi0, lo1, hi1, scale2);
             pv_accumulate<HD, 8>(O, S, sV, 0, lane);
@@ -874,14 +910,17 @@ static cudaError_t launch_cluster(K kernel, dim3 grid, dim3 block, size_t smem, 
 ZI_EXPORT int zi_decode_attention(const void* q, const void* cache, void* out, const int* tables, const int* tok_seg,
                                   const int* pos, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                   int page_size, int max_blocks, long long page_stride, long long kv_stride,
-                                  int window, float scale, const float* sinks, float softcap, cudaStream_t stream) {
+                                  int window, float scale, const float* sinks, float softcap, const float* bias, int bias_len, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (check_common("decode_attention", n_heads, n_kv_heads, head_dim, page_size, max_blocks)) return 1;
+    if (bias && (bias_len <= 0 || !(scale > 0.0f))) return zi_fail("decode_attention: a bias by distance needs a table and a positive scale");
     if (n_tokens > 65535) return zi_fail("decode_attention: %d tokens are more than one launch takes (65535)", n_tokens);
     const int group = n_heads / n_kv_heads, q_blocks = (group + 15) / 16;
     if (n_kv_heads * q_blocks > 65535) return zi_fail("decode_attention: too many head blocks for one launch");
     dim3 grid(DEC_CLUSTER, n_kv_heads * q_blocks, n_tokens);
     const float scale2 = (softcap > 0.0f ? softcap : scale) * LOG2E, cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
+    const DistanceBias db = {bias, bias_len};
+    const float bias_inv = bias ? 1.0f / (softcap > 0.0f ? softcap : scale) : 0.0f;
     const int shift = page_shift_of(page_size);
     cudaError_t e;
     if (head_dim == 128) {
@@ -889,13 +928,13 @@ ZI_EXPORT int zi_decode_attention(const void* q, const void* cache, void* out, c
         if (set_smem(decode_attention_kernel<128>, smem, "decode_attention")) return 1;
         e = launch_cluster(decode_attention_kernel<128>, grid, dim3(ATT_THREADS), smem, stream,
                            (const bf16*)q, (const bf16*)cache, (bf16*)out, tables, tok_seg, pos, n_heads, n_kv_heads,
-                           q_blocks, page_size, shift, max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in);
+                           q_blocks, page_size, shift, max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in, db, bias_inv);
     } else {
         const size_t smem = 16 * 64 * 2 + DEC_STAGES * 2 * TILE_KEYS * 64 * 2 + (32 + 16 * (64 + 8)) * 4;
         if (set_smem(decode_attention_kernel<64>, smem, "decode_attention")) return 1;
         e = launch_cluster(decode_attention_kernel<64>, grid, dim3(ATT_THREADS), smem, stream,
                            (const bf16*)q, (const bf16*)cache, (bf16*)out, tables, tok_seg, pos, n_heads, n_kv_heads,
-                           q_blocks, page_size, shift, max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in);
+                           q_blocks, page_size, shift, max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in, db, bias_inv);
     }
     if (e != cudaSuccess) { cudaGetLastError(); return zi_fail("decode_attention: launch failed: %s", cudaGetErrorString(e)); }
     return zi_check_launch("decode_attention");
@@ -930,6 +969,7 @@ struct DtArgs {
     const CUtensorMap* mkv; const void* q; void* out; const int* tables; const int* tok_seg; const int* pos; int* status;
     int n_tokens, n_heads, n_kv_heads, q_blocks, page_size, box_rows, max_blocks, window; float scale2; cudaStream_t stream;
     int n_splits, min_split_tiles; float* part; int kv_box; const float* sinks; int one_plane; float cap_in;
+    DistanceBias bias; float bias_inv;
 };
 
 template <int HD, int KEYS, int CL>
@@ -952,7 +992,7 @@ static cudaError_t dt_launch(const DtArgs& a) {
     return cudaLaunchKernelEx(&cfg, decode_attention_tma_kernel<HD, KEYS, CL>, *a.mkv, (const bf16*)a.q, (bf16*)a.out, a.tables,
                               a.tok_seg, a.pos, a.status, a.n_heads, a.n_kv_heads, a.q_blocks, a.page_size, a.box_rows,
                               a.max_blocks, a.window, a.scale2, a.n_splits, a.min_split_tiles, a.part, a.kv_box, a.sinks, a.one_plane,
-                              a.cap_in);
+                              a.cap_in, a.bias, a.bias_inv);
 }
 template <int HD>
 static cudaError_t dt_dispatch(const DtArgs& a, int keys, int cl) {
@@ -1022,7 +1062,8 @@ ZI_EXPORT int zi_decode_attention_tma(const void* q, const void* cache, void* ou
                                       const int* pos, int* status, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                       int page_size, int max_blocks, long long n_pages, long long page_stride,
                                       long long kv_stride, int window, float scale, int max_kv_len, float* part,
-                                      long long part_floats, const float* sinks, float softcap, cudaStream_t stream) {
+                                      long long part_floats, const float* sinks, float softcap, const float* bias, int bias_len,
+                                      cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (check_common("decode_attention_tma", n_heads, n_kv_heads, head_dim, page_size, max_blocks)) return 1;
     if (page_size < 8 || page_size > 128 || (page_size & (page_size - 1))) return zi_fail("decode_attention_tma: page size %d is not a power of two from 8 to 128", page_size);
@@ -1030,6 +1071,7 @@ ZI_EXPORT int zi_decode_attention_tma(const void* q, const void* cache, void* ou
     if (((uintptr_t)q | (uintptr_t)cache) & 15) return zi_fail("decode_attention_tma: q and cache must be 16-byte aligned");
     if ((page_stride | kv_stride) & 7) return zi_fail("decode_attention_tma: cache strides must be multiples of 8 elements");
     if (!status) return zi_fail("decode_attention_tma: a status word is required");
+    if (bias && (bias_len <= 0 || !(scale > 0.0f))) return zi_fail("decode_attention_tma: a bias by distance needs a table and a positive scale");
     const int group = n_heads / n_kv_heads, q_blocks = (group + 15) / 16;
     if (tc_init()) return 1;
     DtPlan plan;
@@ -1047,7 +1089,8 @@ ZI_EXPORT int zi_decode_attention_tma(const void* q, const void* cache, void* ou
     if (tc_map_kv_pages(&mkv, cache, head_dim, page_size, n_kv_heads, n_pages, page_stride, kv_stride, box_rows, kv_box ? 2 : 1)) return 1;
     DtArgs a = {&mkv, q, out, tables, tok_seg, pos, status, n_tokens, n_heads, n_kv_heads, q_blocks, page_size, box_rows,
                 max_blocks, window, (softcap > 0.0f ? softcap : scale) * LOG2E, stream, plan.splits, plan.min_split_tiles, part, kv_box,
-                sinks, one_plane, softcap > 0.0f ? scale / softcap : 0.0f};
+                sinks, one_plane, softcap > 0.0f ? scale / softcap : 0.0f, DistanceBias{bias, bias_len},
+                bias ? 1.0f / (softcap > 0.0f ? softcap : scale) : 0.0f};
     cudaError_t e = head_dim == 128 ? dt_dispatch<128>(a, keys, plan.cl) : dt_dispatch<64>(a, keys, plan.cl);
     if (e != cudaSuccess) { cudaGetLastError(); return zi_fail("decode_attention_tma: launch failed: %s", cudaGetErrorString(e)); }
     if (plan.splits > 1) {
@@ -1061,25 +1104,28 @@ ZI_EXPORT int zi_decode_attention_tma(const void* q, const void* cache, void* ou
 ZI_EXPORT int zi_prefill_attention(const void* q, const void* cache, void* out, const int* tables, const int* tiles,
                                    const int* pos, int n_tiles, int n_heads, int n_kv_heads, int head_dim,
                                    int page_size, int max_blocks, long long page_stride, long long kv_stride,
-                                   int window, float scale, const float* sinks, float softcap, cudaStream_t stream) {
+                                   int window, float scale, const float* sinks, float softcap, const float* bias, int bias_len, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (check_common("prefill_attention", n_heads, n_kv_heads, head_dim, page_size, max_blocks)) return 1;
+    if (bias && (bias_len <= 0 || !(scale > 0.0f))) return zi_fail("prefill_attention: a bias by distance needs a table and a positive scale");
     if (n_heads > 65535) return zi_fail("prefill_attention: %d heads are more than one launch takes", n_heads);
     dim3 grid(2 * n_tiles, n_heads);          // two 64-row halves per tile of the list
     const float scale2 = (softcap > 0.0f ? softcap : scale) * LOG2E, cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
+    const DistanceBias db = {bias, bias_len};
+    const float bias_inv = bias ? 1.0f / (softcap > 0.0f ? softcap : scale) : 0.0f;
     const int shift = page_shift_of(page_size);
     if (head_dim == 128) {
         const size_t smem = 5 * TILE_KEYS * 128 * 2;
         if (set_smem(prefill_attention_kernel<128>, smem, "prefill_attention")) return 1;
         prefill_attention_kernel<128><<<grid, ATT_THREADS, smem, stream>>>(
             (const bf16*)q, (const bf16*)cache, (bf16*)out, tables, tiles, pos, n_heads, n_kv_heads, page_size, shift,
-            max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in);
+            max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in, db, bias_inv);
     } else {
         const size_t smem = 5 * TILE_KEYS * 64 * 2;
         if (set_smem(prefill_attention_kernel<64>, smem, "prefill_attention")) return 1;
         prefill_attention_kernel<64><<<grid, ATT_THREADS, smem, stream>>>(
             (const bf16*)q, (const bf16*)cache, (bf16*)out, tables, tiles, pos, n_heads, n_kv_heads, page_size, shift,
-            max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in);
+            max_blocks, page_stride, kv_stride, window, scale2, sinks, cap_in, db, bias_inv);
     }
     return zi_check_launch("prefill_attention");
 }

@@ -109,6 +109,8 @@ struct FaParams {
                                    // scale2 tanh(s cap_in) = log2(e) c tanh(s scale / c)
     const float* sinks;            // optional, one float per query head: exp(sinks[h]) joins the softmax's denominator
     int one_plane;                 // the cache has one plane, whose rows are keys and values at once
+    DistanceBias bias;             // optional: a number per query head and distance joins the score
+    float bias_inv;                // 1 / what multiplies a raw score: the table's numbers are added to raw scores
 };
 
 // TMEM columns of a CTA: two score buffers, the output, and the two A operands (bfloat16 pairs, one row per lane)
@@ -117,7 +119,7 @@ struct FaParams {
 #define FA_COL_Q 384
 #define FA_COL_P 448
 
-template <int HD>
+template <int HD, bool BIAS>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, const FaParams p) {
     constexpr int HH = HD / 64;                               // 64-wide halves of a head
@@ -145,7 +147,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
     const int n0 = p.tiles[tile * 3], rows = p.tiles[tile * 3 + 1], seg = p.tiles[tile * 3 + 2];
     const int h = blockIdx.x, kvh = h / (p.n_heads / p.n_kv_heads);
     const int p0 = p.pos[n0], p_last = p0 + rows - 1;         // positions of a tile are consecutive
-    const int lo_tile = (p.window > 0 && p0 - p.window + 1 > 0) ? p0 - p.window + 1 : 0;
+    const int lo_tile = first_visible_key(p0, p.window);
     const int kt_begin = lo_tile / FA_KEYS, n_kt = p_last / FA_KEYS - kt_begin + 1;
 
     // the softmax warps ask for their 32 rows of Q before anything else, CH requests a lane in flight together
@@ -274,7 +276,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
         // ---- softmax: one thread per query row --------------------------------------------------------------------
         const int quad = warp & 3, r = quad * 32 + lane;
         const int qpos = p0 + r;
-        const int lo = (p.window > 0 && qpos - p.window + 1 > 0) ? qpos - p.window + 1 : 0;
+        const int lo = first_visible_key(qpos, p.window), lo_last = first_visible_key(p_last, p.window);
         const uint32_t lane_base = tmem_base + ((uint32_t)(quad * 32) << 16);
         {   // the rows of Q go through shared memory into TMEM, two bfloat16 per column; rows beyond the tile are zero
 #pragma unroll
@@ -301,8 +303,27 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
         float m_run = -INFINITY, m_used = -INFINITY, l = 0.0f;
         bool ok = true;
         uint32_t s[4][32];
+        // Bias by distance: a tile asks for 159 neighbouring distances of a warp's 32 rows.  They lie in the warp's own stretch
+        // of the row stage, which is free between Q's way in and O's way out, so that lanes read consecutive words; a tile
+        // farther away than the table reaches has one number, which joins the softmax's offset.
+        const float* bias_row = BIAS ? p.bias.table + (size_t)h * p.bias.len : nullptr;
+        float* bias_tab = reinterpret_cast<float*>(stage + quad * 32 * (HD * 2));
         for (int j = 0; j < n_kt; ++j) {
             const int st = j & 1, key0 = (kt_begin + j) * FA_KEYS;
+            const int dist0 = p0 + quad * 32 - key0 - (FA_KEYS - 1);      // the warp's least distance in this tile
+            const bool far = BIAS && dist0 >= p.bias.len - 1;
+            float off2 = 0.0f;
+            if (BIAS) {
+                if (far) {
+                    off2 = __ldg(bias_row + p.bias.len - 1) * 1.4426950408889634f;
+                } else {
+                    __syncwarp();                                         // the tile before has been read
+#pragma unroll
+                    for (int i = 0; i < 5; ++i)
+                        bias_tab[i * 32 + lane] = __ldg(bias_row + min(max(dist0 + i * 32 + lane, 0), p.bias.len - 1)) * p.bias_inv;
+                    __syncwarp();
+                }
+            }
             if (!mbar_wait_warp(s_full + 8 * st, (j >> 1) & 1, &gave_up)) { ok = false; break; }
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
 #pragma unroll
@@ -320,8 +341,15 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
                         s[q4][c] = __float_as_uint(1.0f - __fdividef(2.0f, 1.0f + fa_exp2(y * 2.8853900817779268f)));
                     }
             }
+            if (BIAS && !far) {
+#pragma unroll
+                for (int q4 = 0; q4 < 4; ++q4)
+#pragma unroll
+                    for (int c = 0; c < 32; ++c)
+                        s[q4][c] = __float_as_uint(__uint_as_float(s[q4][c]) + bias_tab[lane + FA_KEYS - 1 - q4 * 32 - c]);
+            }
             // keys this row must not see; whole tiles below the diagonal and inside the window need no test
-            const bool need_mask = key0 + FA_KEYS - 1 > p0 || (p.window > 0 && key0 < p_last - p.window + 1);
+            const bool need_mask = key0 + FA_KEYS - 1 > p0 || key0 < lo_last;
             if (need_mask) {
 #pragma unroll
                 for (int q4 = 0; q4 < 4; ++q4)
@@ -338,7 +366,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
                 for (int c = 0; c < 32; c += 2)
                     mx[(c >> 1) & 3] = fa_max3(mx[(c >> 1) & 3], __uint_as_float(s[q4][c]), __uint_as_float(s[q4][c + 1]));
             const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-            const float m_new = fmaxf(m_run, m_tile * p.scale2);
+            const float m_new = fmaxf(m_run, BIAS ? fmaf(m_tile, p.scale2, off2) : m_tile * p.scale2);
             const bool grow = m_new > m_used + FA_LAZY_LOG2;            // false while both are -inf
             const bool any_grow = __any_sync(0xffffffffu, grow);
             const float f = grow ? fa_exp2(m_used - m_new) : 1.0f;      // 0 when nothing was seen before
@@ -347,7 +375,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
             const float mu = m_used == -INFINITY ? 0.0f : m_used;       // nothing seen yet: every p is exp2(-inf) = 0
             uint64_t sums2[2] = {0ull, 0ull};                            // two pairs of partial sums
             uint32_t pk[2][32];                                          // the row of P, two bfloat16 per word
-            const uint64_t scale22 = f2_pack(p.scale2, p.scale2), nmu2 = f2_pack(-mu, -mu), magic2 = f2_pack(12582912.0f, 12582912.0f);
+            const uint64_t scale22 = f2_pack(p.scale2, p.scale2), nmu2 = BIAS ? f2_pack(off2 - mu, off2 - mu) : f2_pack(-mu, -mu), magic2 = f2_pack(12582912.0f, 12582912.0f);
             const uint64_t c3 = f2_pack(0.055171459913253784f, 0.055171459913253784f), c2 = f2_pack(0.2426108568906784f, 0.2426108568906784f),
                            c1 = f2_pack(0.6932609677314758f, 0.6932609677314758f), c0 = f2_pack(0.9999281167984009f, 0.9999281167984009f);
 #pragma unroll
@@ -441,6 +469,14 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, con
     }
 }
 
+template <int HD, bool BIAS>
+static int fa_launch(const CUtensorMap& mkv, const FaParams& p, dim3 grid, size_t smem, cudaStream_t stream) {
+    const cudaError_t e = cudaFuncSetAttribute(prefill_attention_tcgen05_kernel<HD, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return zi_fail("prefill_attention_tcgen05: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+    prefill_attention_tcgen05_kernel<HD, BIAS><<<grid, FA_THREADS, smem, stream>>>(mkv, p);
+    return 0;
+}
+
 // ---- host side -----------------------------------------------------------------------------------------
 // tiles: int32 [n_tiles, 3] = (first token, rows <= 128, segment).  status: one int of device memory, zero before;
 // non-zero afterwards means a bounded wait ran out (11 producer, 12/13 MMA issuer, 14 softmax).
@@ -448,7 +484,7 @@ ZI_EXPORT int zi_prefill_attention_tcgen05(const void* q, const void* cache, voi
                                            const int* pos, int* status, int n_tokens, int n_tiles, int n_heads, int n_kv_heads,
                                            int head_dim, int page_size, int max_blocks, long long n_pages, long long page_stride,
                                            long long kv_stride, int window, float scale, const float* sinks,
-                                           float softcap, cudaStream_t stream) {
+                                           float softcap, const float* bias, int bias_len, cudaStream_t stream) {
     if (n_tiles <= 0 || n_tokens <= 0) return 0;
     if (head_dim != 64 && head_dim != 128) return zi_fail("prefill_attention_tcgen05: head_dim %d is not 64 or 128", head_dim);
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads) return zi_fail("prefill_attention_tcgen05: %d heads over %d key-value heads", n_heads, n_kv_heads);
@@ -457,6 +493,7 @@ ZI_EXPORT int zi_prefill_attention_tcgen05(const void* q, const void* cache, voi
     if (((uintptr_t)q | (uintptr_t)cache | (uintptr_t)out) & 15) return zi_fail("prefill_attention_tcgen05: q, cache and out must be 16-byte aligned");
     if ((page_stride | kv_stride) & 7) return zi_fail("prefill_attention_tcgen05: cache strides must be multiples of 8 elements");
     if (!status) return zi_fail("prefill_attention_tcgen05: a status word is required");
+    if (bias && (bias_len <= 0 || !(scale > 0.0f))) return zi_fail("prefill_attention_tcgen05: a bias by distance needs a table and a positive scale");
     if (tc_init()) return 1;
     CUtensorMap mkv;
     if (tc_map_kv_pages(&mkv, cache, head_dim, page_size, n_kv_heads, n_pages, page_stride, kv_stride, page_size)) return 1;
@@ -466,17 +503,14 @@ ZI_EXPORT int zi_prefill_attention_tcgen05(const void* q, const void* cache, voi
     p.scale2 = (softcap > 0.0f ? softcap : scale) * 1.4426950408889634f;
     p.cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
     p.sinks = sinks; p.one_plane = kv_stride == 0 ? 1 : 0;
+    p.bias = DistanceBias{bias, bias_len};
+    p.bias_inv = bias ? 1.0f / (softcap > 0.0f ? softcap : scale) : 0.0f;
     const dim3 grid(n_heads, n_tiles);
     const size_t smem = (size_t)FA_STAGE_OFFSET(head_dim) + (size_t)FA_ROWS * head_dim * 2;
-    cudaError_t e;
     if (head_dim == 128) {
-        e = cudaFuncSetAttribute(prefill_attention_tcgen05_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return zi_fail("prefill_attention_tcgen05: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
-        prefill_attention_tcgen05_kernel<128><<<grid, FA_THREADS, smem, stream>>>(mkv, p);
+        if (bias ? fa_launch<128, true>(mkv, p, grid, smem, stream) : fa_launch<128, false>(mkv, p, grid, smem, stream)) return 1;
     } else {
-        e = cudaFuncSetAttribute(prefill_attention_tcgen05_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return zi_fail("prefill_attention_tcgen05: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
-        prefill_attention_tcgen05_kernel<64><<<grid, FA_THREADS, smem, stream>>>(mkv, p);
+        if (bias ? fa_launch<64, true>(mkv, p, grid, smem, stream) : fa_launch<64, false>(mkv, p, grid, smem, stream)) return 1;
     }
     return zi_check_launch("prefill_attention_tcgen05");
 }

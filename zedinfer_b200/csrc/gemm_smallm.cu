@@ -142,7 +142,7 @@ __device__ __forceinline__ void accumulate_rows(float (&acc)[NT][4], const bf16*
 
 // What the epilogue does to the sums.  kind 0: the template's own rule (SILU_MUL: up * silu(gate); else + bias);
 // kind 2 (with SILU_MUL, W = [gate; up]): g = min(gate, limit), u = clamp(up, -limit, limit) (limit <= 0: no clamps),
-// g * sigmoid(slope * g) * (u + up_offset); kind 3 (without): max(x, 0)^2.
+// g * sigmoid(slope * g) * (u + up_offset); kind 3 (without): max(x, 0)^2; kind 4 (with SILU_MUL): gelu_tanh(gate) * up.
 struct GsAct { int kind; float limit, slope, up_offset; };
 
 template <int NT, typename TC, bool SILU_MUL>
@@ -249,6 +249,8 @@ gemm_smallm_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, const
                 float g2 = gr, u2 = ur;
                 if (act.limit > 0.0f) { g2 = fminf(g2, act.limit); u2 = fminf(fmaxf(u2, -act.limit), act.limit); }
                 v = (g2 / (1.0f + expf(-act.slope * g2))) * (u2 + act.up_offset);
+            } else if (act.kind == 4) {
+                v = gelu_tanh(gr) * ur;
             } else {
                 v = ur * gr / (1.0f + expf(-gr));
             }
@@ -315,10 +317,10 @@ ZI_EXPORT int zi_gemm_smallm(const void* X, const void* W, const void* bias, voi
                              int* counters, int M, int N, int K, long long ldx, long long ldw, long long ldc,
                              int silu_mul, int act_kind, float act_limit, float act_slope, float act_offset,
                              cudaStream_t stream) {
-    // act_kind: see GsAct (2 needs silu_mul's stacked weight, 3 a plain product without bias)
+    // act_kind: see GsAct (2 and 4 need silu_mul's stacked weight, 3 a plain product without bias)
     if (M <= 0 || N <= 0) return 0;
     if (M > 16) return zi_fail("gemm_smallm: M=%d rows; this kernel takes at most 16", M);
-    if ((act_kind == 2 && !silu_mul) || (act_kind == 3 && (silu_mul || bias)) || (act_kind != 0 && act_kind != 2 && act_kind != 3))
+    if (((act_kind == 2 || act_kind == 4) && !silu_mul) || (act_kind == 3 && (silu_mul || bias)) || act_kind < 0 || act_kind == 1 || act_kind > 4)
         return zi_fail("gemm_smallm: activation %d does not fit this product", act_kind);
     const GsAct act = {act_kind, act_limit, act_slope, act_offset};
     if (K <= 0 || K % 32 != 0) return zi_fail("gemm_smallm: K=%d must be a positive multiple of 32", K);

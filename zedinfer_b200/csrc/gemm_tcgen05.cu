@@ -179,7 +179,7 @@ struct TpParams {
     int M, N, K;                // N: columns of C (silu_mul: the intermediate size)
     int c_is_f32, silu_mul;
     int act;                    // 1: up * silu(gate); 2: the clamped, sigmoid-gated product (both with silu_mul's stacked
-    float act_limit, act_slope, act_offset;   // weight); 3: max(x, 0)^2 on a plain product; 0: nothing
+    float act_limit, act_slope, act_offset;   // weight); 3: max(x, 0)^2 on a plain product; 4: up * gelu_tanh(gate); 0: nothing
     int bn;                     // accumulator columns per tile
     int up_row0;                // silu_mul: first row of the up half in W
     int tiles_m, tiles_n;
@@ -236,6 +236,11 @@ __device__ __forceinline__ void tp_epilogue_row(const TpParams& p, uint32_t tadd
                             uv = __bfloat162float(__float2bfloat16_rn(uv));
                             if (p.act_limit > 0.0f) { gv = fminf(gv, p.act_limit); uv = fminf(fmaxf(uv, -p.act_limit), p.act_limit); }
                             v[j] = __fdividef(gv, 1.0f + __expf(-p.act_slope * gv)) * (uv + p.act_offset);
+                        } else if (p.act == 4) {
+                            // rounded as above; (1 + tanh(y)) / 2 = 1 / (1 + exp(-2 y))
+                            gv = __bfloat162float(__float2bfloat16_rn(gv));
+                            uv = __bfloat162float(__float2bfloat16_rn(uv));
+                            v[j] = __fdividef(gv, 1.0f + __expf(-2.0f * GELU_TANH_SLOPE * gv * fmaf(GELU_TANH_CUBIC * gv, gv, 1.0f))) * uv;
                         } else {
                             v[j] = __fdividef(gv, 1.0f + __expf(-gv)) * uv;
                         }
@@ -602,18 +607,19 @@ static int tp_step_cost(int bn) { const int pipe = bn / 2, smem = 32 + bn / 4; r
 // C[M,N] = X[M,K] . W^T with the persistent kernel.  epilogue 0: W is [N,K], optional bias[N].
 // epilogue 1 (silu_mul): W is [2N,K] = [gate; up], C = silu(X.gate^T) * (X.up^T), no bias.
 // epilogue 2: the same stacked weight, C = g * sigmoid(slope * g) * (u + offset) with g = min(gate, limit), u = clamp(up,
-// -limit, limit) (limit <= 0: no clamps); epilogue 3: W is [N,K], C = max(X.W^T, 0)^2, no bias.
+// -limit, limit) (limit <= 0: no clamps); epilogue 3: W is [N,K], C = max(X.W^T, 0)^2, no bias;
+// epilogue 4: the stacked weight again, C = gelu_tanh(X.gate^T) * (X.up^T).
 // bn_hint: 0 lets the call choose the tile width; else a multiple of 16 (32 for silu_mul) up to 256.
 ZI_EXPORT int zi_gemm_tcgen05_tiles(const void* X, const void* W, const void* bias, void* C, int c_dtype, int* status, int M, int N,
                                     int K, long long ldx, long long ldw, long long ldc, int epilogue, int bn_hint, int num_sms,
                                     float act_limit, float act_slope, float act_offset, cudaStream_t stream) {
-    const bool gated = epilogue == 1 || epilogue == 2;
+    const bool gated = epilogue == 1 || epilogue == 2 || epilogue == 4;
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0) return zi_fail("gemm_tcgen05: K=%d must be positive", K);
     if (K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return zi_fail("gemm_tcgen05: K and the row strides must be multiples of 8 elements (16 bytes) for TMA; got K=%d ldx=%lld ldw=%lld", K, ldx, ldw);
     if (((uintptr_t)X | (uintptr_t)W) & 15) return zi_fail("gemm_tcgen05: operands must be 16-byte aligned");
     if (c_dtype != ZI_F32 && c_dtype != ZI_BF16) return zi_fail("gemm_tcgen05: unknown output dtype %d", c_dtype);
-    if (epilogue < 0 || epilogue > 3) return zi_fail("gemm_tcgen05: unknown epilogue %d", epilogue);
+    if (epilogue < 0 || epilogue > 4) return zi_fail("gemm_tcgen05: unknown epilogue %d", epilogue);
     if (epilogue != 0 && bias) return zi_fail("gemm_tcgen05: the silu_mul epilogue takes no bias");
     if (!status) return zi_fail("gemm_tcgen05: a status word is required");
     if (num_sms <= 0) return zi_fail("gemm_tcgen05: num_sms=%d must be positive", num_sms);
@@ -660,13 +666,13 @@ ZI_EXPORT int zi_gemm_tcgen05_tiles(const void* X, const void* W, const void* bi
 ZI_EXPORT int zi_gemm_tcgen05_grouped(const void* X, const void* W, void* C, int c_dtype, int* status, int M, int N, int K,
                                       long long ldx, long long ldc, int epilogue, int n_experts, const int* tile_expert,
                                       int num_sms, float act_limit, float act_slope, float act_offset, cudaStream_t stream) {
-    const bool gated = epilogue == 1 || epilogue == 2;
+    const bool gated = epilogue == 1 || epilogue == 2 || epilogue == 4;
     if (M <= 0 || N <= 0) return 0;
     if (M % TC_BM) return zi_fail("gemm_tcgen05_grouped: M=%d must be a multiple of %d", M, TC_BM);
     if (K <= 0 || K % 8 != 0 || ldx % 8 != 0) return zi_fail("gemm_tcgen05_grouped: K=%d and ldx=%lld must be positive multiples of 8", K, ldx);
     if (((uintptr_t)X | (uintptr_t)W) & 15) return zi_fail("gemm_tcgen05_grouped: operands must be 16-byte aligned");
     if (c_dtype != ZI_F32 && c_dtype != ZI_BF16) return zi_fail("gemm_tcgen05_grouped: unknown output dtype %d", c_dtype);
-    if (epilogue < 0 || epilogue > 3) return zi_fail("gemm_tcgen05_grouped: unknown epilogue %d", epilogue);
+    if (epilogue < 0 || epilogue > 4) return zi_fail("gemm_tcgen05_grouped: unknown epilogue %d", epilogue);
     if (!status || !tile_expert || n_experts <= 0 || num_sms <= 0) return zi_fail("gemm_tcgen05_grouped: status, tile_expert, experts and num_sms are required");
     if (tc_init()) return 1;
     const int step = gated ? 32 : 16;
@@ -710,13 +716,13 @@ static int tq_step_cost(int bn) { const int pipe = bn / 2, smem = 32 + bn / 8; r
 ZI_EXPORT int zi_gemm_tcgen05_pairs(const void* X, const void* W, const void* bias, void* C, int c_dtype, int* status, int M, int N,
                                     int K, long long ldx, long long ldw, long long ldc, int epilogue, int bn_hint,
                                     float act_limit, float act_slope, float act_offset, cudaStream_t stream) {
-    const bool gated = epilogue == 1 || epilogue == 2;
+    const bool gated = epilogue == 1 || epilogue == 2 || epilogue == 4;
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0) return zi_fail("gemm_tcgen05: K=%d must be positive", K);
     if (K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return zi_fail("gemm_tcgen05: K and the row strides must be multiples of 8 elements (16 bytes) for TMA; got K=%d ldx=%lld ldw=%lld", K, ldx, ldw);
     if (((uintptr_t)X | (uintptr_t)W) & 15) return zi_fail("gemm_tcgen05: operands must be 16-byte aligned");
     if (c_dtype != ZI_F32 && c_dtype != ZI_BF16) return zi_fail("gemm_tcgen05: unknown output dtype %d", c_dtype);
-    if (epilogue < 0 || epilogue > 3) return zi_fail("gemm_tcgen05: unknown epilogue %d", epilogue);
+    if (epilogue < 0 || epilogue > 4) return zi_fail("gemm_tcgen05: unknown epilogue %d", epilogue);
     if (epilogue != 0 && bias) return zi_fail("gemm_tcgen05: the silu_mul epilogue takes no bias");
     if (!status) return zi_fail("gemm_tcgen05: a status word is required");
     if (tc_init()) return 1;

@@ -1,6 +1,6 @@
 // Linear recurrences with a matrix state per head, over the tokens of one step:
 //
-//   zi_linear_state         per head a state S (dim x vdim, float32) walked token by token in one of two rules:
+//   zi_linear_state         per head a state S (dim x vdim, float32) walked token by token in one of four rules:
 //                             delta  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //                                    with q, k made unit vectors per head (q also times q_scale), beta = sigmoid(b) and a
 //                                    decay per head and key entry g = exp(-exp(A_log) softplus(a + dt_bias))
@@ -9,14 +9,20 @@
 //                             forget S <- diag(f) S + (1 - f) v^T;  o = S^T q   with the gate per head and key entry
 //                                    f = l + (1 - l) sigmoid(a), l a lower bound per head and key entry; 1 - f stands
 //                                    where the other rules have a key
+//                             expgate S <- F S + I k v^T;  n <- F n + I k;  o = S^T q,  den = max(|n . q|, exp(-m)) + 1e-6
+//                                    with exponential gates kept in range by a running maximum m of their logarithms:
+//                                    i = c tanh((a + bi) / c), f = ln sigmoid(c tanh((b + bf) / c)) per head, m' = max(f + m, i)
+//                                    (m = 0 before the first token), F = exp(f + m - m'), I = exp(i - m')
 //                           the state read from and written back to the request's slot
-//   zi_group_rmsnorm_gate   out = unit_rms_per_group(y) * w * gate(z), the gate sigmoid, SiLU or none
+//   zi_group_rmsnorm_gate   out = unit_rms_per_group(y / den) * w * gate(z), the gate sigmoid, SiLU or none, den optional
 //
 // Everything that enters the recurrence is float32: unit vectors, sigmoid, softplus, exponentials, decays, the state,
 // the sums.  A token's sums have one order that depends on the sizes alone, and tokens are walked one by one, so a token's
 // result does not depend on how its request was cut into steps or on what else is in the batch.
 //
-// A request's state slot (float32) holds S laid out [heads, vdim, dim]: a column's key entries are consecutive.  Slot -1
+// A request's state slot (float32) holds S laid out [heads, vdim, dim]: a column's key entries are consecutive.  The expgate
+// rule has one column more, n (what a value of 1 would leave in S), and m behind the columns, once per column so that the
+// blocks that share a head never wait for one another: [heads, vdim + 1, dim], then [heads, vdim + 1].  Slot -1
 // (a row of padding): the state is zero and nothing is written.
 #include "zi_common.cuh"
 
@@ -32,16 +38,18 @@ ZI_DEFINE_LAST_ERROR(linrec)
 struct LinearStateArgs {
     const void* q; const void* k; const void* v; const void* a; const void* b;
     long long ldq, ldk, ldv, lda, ldb;
-    const float* dt_bias;        // [heads * dim]   (delta; forget: the gates' lower bounds)
-    const float* a_log;          // [heads]         (delta)
+    const float* dt_bias;        // [heads * dim]   (delta; forget: the gates' lower bounds; expgate: bi [heads])
+    const float* a_log;          // [heads]         (delta; expgate: bf)
     const float* decay;          // [heads]         (decay)
     float* state; long long slot_stride;
     const int* slots; const int* bounds;
     float* y;                    // [tokens, heads * vdim]
+    float* den;                  // [tokens, heads] (expgate): what the read-out is to be divided by
     int n_segments, heads, kv_heads, dim, vdim;
     int act_silu;                // bit 0: SiLU on q, bit 1: on k, bit 2: on v
     int decay_per_head;          // delta: a is [tokens, heads] and dt_bias [heads]: one decay per head instead of one per key entry
     float q_scale, unit_eps;
+    float gate_cap;              // c (expgate)
 };
 
 // The rules: which of them keeps a decay per key entry in a token's record, and which corrects the write by what the state
@@ -49,7 +57,10 @@ struct LinearStateArgs {
 #define LR_DELTA 0
 #define LR_DECAY 1
 #define LR_FORGET 2
-#define LR_PER_ENTRY(RULE) ((RULE) != LR_DECAY)
+#define LR_EXPGATE 3
+#define LR_PER_ENTRY(RULE) ((RULE) == LR_DELTA || (RULE) == LR_FORGET)
+#define LR_COLUMNS(RULE, vdim) ((RULE) == LR_EXPGATE ? (vdim) + 1 : (vdim))    // columns of S in a head's state
+#define LR_DEN_EPS 1e-6f
 
 __device__ __forceinline__ float lr_softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float lr_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -91,6 +102,21 @@ __device__ __forceinline__ float lr_ready_qk(const T* __restrict__ qr, const T* 
 
 // The decay of one head and key entry: exp(-rate softplus(a + dt_bias)).
 __device__ __forceinline__ float lr_decay(float a, float dt_bias, float rate) { return expf(-rate * lr_softplus(a + dt_bias)); }
+
+// The logarithms of a token's gates of one head (expgate), from their projections.
+__device__ __forceinline__ float lr_log_input_gate(float a, float bias, float cap) { return cap * tanhf((a + bias) / cap); }
+__device__ __forceinline__ float lr_log_forget_gate(float b, float bias, float cap) {
+    const float z = cap * tanhf((b + bias) / cap);
+    return fminf(z, 0.0f) - log1pf(expf(-fabsf(z)));
+}
+// One token's step of the running maximum: m becomes max(f + m, i); one of fade and write is exp(0).
+__device__ __forceinline__ void lr_gate_step(float& m, float i, float f, float& fade, float& write) {
+    const float fm = f + m, d = fm - i;
+    const float e = expf(-fabsf(d));
+    fade = d < 0.0f ? e : 1.0f;
+    write = d < 0.0f ? 1.0f : e;
+    m = fmaxf(fm, i);
+}
 
 // One warp makes everything ready that token n brings to head h's walk besides its values: query dq, key dk and, where the
 // rule keeps one per key entry, decays dg (DP floats each, zero past dim).  Returns q . k.  rate: exp(A_log) of the head.
@@ -201,6 +227,13 @@ __device__ __forceinline__ float lr_walk_token(float (&S)[R], const float* sk, c
     return fmaf(qk, u, qs);
 }
 
+// A column's output of one token: the read-out, or (expgate, column vdim) the divisor of the head's read-outs.
+template <int RULE>
+__device__ __forceinline__ void lr_emit(const LinearStateArgs& p, size_t n, int h, int col, float o, float m) {
+    if (col < p.vdim) p.y[n * ((size_t)p.heads * p.vdim) + (size_t)h * p.vdim + col] = o;
+    else if (RULE == LR_EXPGATE && col == p.vdim) p.den[n * p.heads + h] = fmaxf(fabsf(o), expf(-m)) + LR_DEN_EPS;
+}
+
 // ---- the walk that makes its own inputs ready (steps of single tokens) -----------------------------------------------------
 // DP = LANES * R >= dim; what lies past dim is zero.
 template <typename T, int R, int LANES, int COLS, int RULE>
@@ -214,11 +247,13 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
     float* sv = sg + (LR_PER_ENTRY(RULE) ? LR_CHUNK * DP : 0);  // [LR_CHUNK][COLS]
     float* sbeta = sv + LR_CHUNK * COLS;        // [LR_CHUNK]
     float* sqk = sbeta + LR_CHUNK;                 // [LR_CHUNK]
+    float* sfg = sqk + LR_CHUNK;                   // [LR_CHUNK]   (expgate)
     const int seg = blockIdx.x / tiles, tile = blockIdx.x - seg * tiles, h = blockIdx.y;
     const int kvh = h / (p.heads / p.kv_heads);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = threadIdx.x % LANES;
     const int col = tile * COLS + threadIdx.x / LANES;
-    const bool live = col < p.vdim;
+    const int columns = LR_COLUMNS(RULE, p.vdim);
+    const bool live = col < columns;
     const int t0 = p.bounds ? p.bounds[2 * seg] : seg, t1 = p.bounds ? p.bounds[2 * seg + 1] : seg + 1;
     const int slot = p.slots[seg];
     const int dim = p.dim, vdim = p.vdim;
@@ -226,7 +261,7 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
     const T* b = (const T*)p.b;
 
     float S[R];
-    float* srow = (slot >= 0 && live) ? p.state + (size_t)slot * p.slot_stride + ((size_t)h * vdim + col) * dim : nullptr;
+    float* srow = (slot >= 0 && live) ? p.state + (size_t)slot * p.slot_stride + ((size_t)h * columns + col) * dim : nullptr;
 #pragma unroll
     for (int i = 0; i < R / 4; ++i)
 #pragma unroll
@@ -236,6 +271,8 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
         }
     const float lam = RULE == LR_DECAY ? p.decay[h] : 0.0f;
     const float rate = RULE == LR_DELTA ? expf(p.a_log[h]) : 0.0f;
+    float* smax = RULE == LR_EXPGATE && srow ? p.state + (size_t)slot * p.slot_stride + (size_t)p.heads * columns * dim + (size_t)h * columns + col : nullptr;
+    float m = smax ? *smax : 0.0f;
 
     for (int c0 = t0; c0 < t1; c0 += LR_CHUNK) {
         const int cnt = min(LR_CHUNK, t1 - c0);
@@ -246,23 +283,35 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
             const float dot = lr_ready_token<T, DP, RULE>(p, n, h, kvh, rate, lane, sq + tt * DP, sk + tt * DP, sg + tt * DP);
             if (lane == 0) {
                 sqk[tt] = dot;
-                sbeta[tt] = RULE == LR_DELTA ? lr_sigmoid(to_f32<T>(b[n * p.ldb + h])) : 1.0f;
+                if (RULE == LR_EXPGATE) {
+                    sbeta[tt] = lr_log_input_gate(to_f32<T>(((const T*)p.a)[n * p.lda + h]), p.dt_bias[h], p.gate_cap);
+                    sfg[tt] = lr_log_forget_gate(to_f32<T>(b[n * p.ldb + h]), p.a_log[h], p.gate_cap);
+                } else {
+                    sbeta[tt] = RULE == LR_DELTA ? lr_sigmoid(to_f32<T>(b[n * p.ldb + h])) : 1.0f;
+                }
             }
         }
         for (int idx = threadIdx.x; idx < cnt * COLS; idx += NT) {
             const int tt = idx / COLS, c = tile * COLS + (idx - tt * COLS);
             float x = c < vdim ? to_f32<T>(v[(size_t)(c0 + tt) * p.ldv + (size_t)h * vdim + c]) : 0.0f;
             if (p.act_silu & 4) x = lr_silu(x);
+            if (RULE == LR_EXPGATE && c == vdim) x = 1.0f;
             sv[idx] = x;
         }
         __syncthreads();
         // ---- walk
         for (int tt = 0; tt < cnt; ++tt) {
-            const float o = lr_walk_token<R, LANES, RULE>(S, sk + tt * DP, sq + tt * DP, sg + tt * DP, lam, sv[tt * COLS + threadIdx.x / LANES],
-                                                           sbeta[tt], sqk[tt], sub);
-            if (sub == 0 && live) p.y[(size_t)(c0 + tt) * ((size_t)p.heads * vdim) + (size_t)h * vdim + col] = o;
+            float fade = lam, vv = sv[tt * COLS + threadIdx.x / LANES];
+            if (RULE == LR_EXPGATE) {
+                float write;
+                lr_gate_step(m, sbeta[tt], sfg[tt], fade, write);
+                vv *= write;
+            }
+            const float o = lr_walk_token<R, LANES, RULE>(S, sk + tt * DP, sq + tt * DP, sg + tt * DP, fade, vv, sbeta[tt], sqk[tt], sub);
+            if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt), h, col, o, m);
         }
     }
+    if (smax && sub == 0) *smax = m;
     if (srow) {
 #pragma unroll
         for (int i = 0; i < R / 4; ++i)
@@ -276,8 +325,8 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
 
 template <typename T, int R, int LANES, int COLS, int RULE>
 static int launch_linear_state(const LinearStateArgs& p, cudaStream_t stream) {
-    const int tiles = (p.vdim + COLS - 1) / COLS;
-    const size_t smem = ((size_t)LR_CHUNK * LANES * R * (LR_PER_ENTRY(RULE) ? 3 : 2) + LR_CHUNK * COLS + 2 * LR_CHUNK) * sizeof(float);
+    const int tiles = (LR_COLUMNS(RULE, p.vdim) + COLS - 1) / COLS;
+    const size_t smem = ((size_t)LR_CHUNK * LANES * R * (LR_PER_ENTRY(RULE) ? 3 : 2) + LR_CHUNK * COLS + 3 * LR_CHUNK) * sizeof(float);
     if (smem > 48 * 1024) {
         static bool raised = false;       // per instantiation
         if (!raised) {
@@ -292,7 +341,7 @@ static int launch_linear_state(const LinearStateArgs& p, cudaStream_t stream) {
 // ---- the walk over inputs made ready beforehand (steps that bring portions of prompts) ---------------------------------
 // Making a token ready (loads from global memory, unit vectors, softplus and exponentials) does not depend on the state, so
 // for long segments it runs first, over all tokens and heads at once, and leaves per token and head one record of float32
-//   [ q DP | k DP | g DP (rules with a decay per key entry) | beta, q . k, 0, 0 ]
+//   [ q DP | k DP | g DP (rules with a decay per key entry) | beta, q . k, 0, 0 ]     (expgate: i, q . k, f, 0)
 // and the values [tiles * COLS] (SiLU applied where asked, zero past vdim).  The walk then only copies records into
 // shared memory, two chunks in flight, and walks.  Both forms call the same functions on a token, so its result has the
 // same bits in either.
@@ -314,11 +363,17 @@ linear_state_ready_kernel(const LinearStateArgs p, float* __restrict__ rec, floa
     const float dot = lr_ready_token<T, DP, RULE>(p, n, h, kvh, rate, lane, r, r + DP, r + 2 * DP);
     float beta = 1.0f;
     if (RULE == LR_DELTA) beta = lr_sigmoid(to_f32<T>(((const T*)p.b)[n * p.ldb + h]));
-    if (lane < 4) r[REC - 4 + lane] = lane == 0 ? beta : (lane == 1 ? dot : 0.0f);
+    float fg = 0.0f;
+    if (RULE == LR_EXPGATE) {
+        beta = lr_log_input_gate(to_f32<T>(((const T*)p.a)[n * p.lda + h]), p.dt_bias[h], p.gate_cap);
+        fg = lr_log_forget_gate(to_f32<T>(((const T*)p.b)[n * p.ldb + h]), p.a_log[h], p.gate_cap);
+    }
+    if (lane < 4) r[REC - 4 + lane] = lane == 0 ? beta : (lane == 1 ? dot : (lane == 2 ? fg : 0.0f));
     float* vr = pv + (size_t)pair * vp;
     for (int c = lane; c < vp; c += 32) {
         float x = c < vdim ? to_f32<T>(v[n * p.ldv + (size_t)h * vdim + c]) : 0.0f;
         if (p.act_silu & 4) x = lr_silu(x);
+        if (RULE == LR_EXPGATE && c == vdim) x = 1.0f;
         vr[c] = x;
     }
 }
@@ -337,13 +392,14 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
     const int seg = blockIdx.x / tiles, tile = blockIdx.x - seg * tiles, h = blockIdx.y;
     const int sub = threadIdx.x % LANES;
     const int col = tile * COLS + threadIdx.x / LANES;
-    const bool live = col < p.vdim;
+    const int columns = LR_COLUMNS(RULE, p.vdim);
+    const bool live = col < columns;
     const int t0 = p.bounds ? p.bounds[2 * seg] : seg, t1 = p.bounds ? p.bounds[2 * seg + 1] : seg + 1;
     const int slot = p.slots[seg];
     const int dim = p.dim, vdim = p.vdim, vp = tiles * COLS;
 
     float S[R];
-    float* srow = (slot >= 0 && live) ? p.state + (size_t)slot * p.slot_stride + ((size_t)h * vdim + col) * dim : nullptr;
+    float* srow = (slot >= 0 && live) ? p.state + (size_t)slot * p.slot_stride + ((size_t)h * columns + col) * dim : nullptr;
 #pragma unroll
     for (int i = 0; i < R / 4; ++i)
 #pragma unroll
@@ -352,6 +408,8 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
             S[i * 4 + e] = (srow && d < dim) ? srow[d] : 0.0f;
         }
     const float lam = RULE == LR_DECAY ? p.decay[h] : 0.0f;
+    float* smax = RULE == LR_EXPGATE && srow ? p.state + (size_t)slot * p.slot_stride + (size_t)p.heads * columns * dim + (size_t)h * columns + col : nullptr;
+    float m = smax ? *smax : 0.0f;
 
     auto fetch = [&](int c0, float* dst) {
         const int cnt = min(LR_WALK_CHUNK, t1 - c0);
@@ -379,17 +437,22 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
         __syncthreads();                                                   // everyone's copies of this chunk have landed
         const float* st = smem + s * STAGE;
         const float* sv = st + LR_WALK_CHUNK * REC + threadIdx.x / LANES;
-        float* yc = p.y + (size_t)c0 * ((size_t)p.heads * vdim) + (size_t)h * vdim + col;
         int tt = 0;
         // four tokens at a time, in straight-line code
         for (; tt + 4 <= cnt; tt += 4) {
-            float qs[4], u[4], qk[4];
+            float qs[4], u[4], qk[4], mt[4];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float* r = st + (tt + j) * REC;
-                float kr[R], ks;
-                lr_token_local<R, LANES, RULE>(S, kr, r + DP, r, r + 2 * DP, lam, sub, ks, qs[j]);
+                float kr[R], ks, fade = lam;
                 u[j] = sv[(tt + j) * COLS];
+                if (RULE == LR_EXPGATE) {
+                    float write;
+                    lr_gate_step(m, r[REC - 4], r[REC - 2], fade, write);
+                    u[j] *= write;
+                }
+                mt[j] = m;
+                lr_token_local<R, LANES, RULE>(S, kr, r + DP, r, r + 2 * DP, fade, sub, ks, qs[j]);
                 qk[j] = r[REC - 3];
                 if (RULE == LR_DELTA) {
 #pragma unroll
@@ -404,15 +467,22 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
                 for (int j = 0; j < 4; ++j) qs[j] += __shfl_xor_sync(0xffffffffu, qs[j], o);
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-                if (sub == 0 && live) yc[(size_t)(tt + j) * ((size_t)p.heads * vdim)] = fmaf(qk[j], u[j], qs[j]);
+                if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt + j), h, col, fmaf(qk[j], u[j], qs[j]), mt[j]);
         }
         for (; tt < cnt; ++tt) {
             const float* r = st + tt * REC;
-            const float o = lr_walk_token<R, LANES, RULE>(S, r + DP, r, r + 2 * DP, lam, sv[tt * COLS], r[REC - 4], r[REC - 3], sub);
-            if (sub == 0 && live) yc[(size_t)tt * ((size_t)p.heads * vdim)] = o;
+            float fade = lam, vv = sv[tt * COLS];
+            if (RULE == LR_EXPGATE) {
+                float write;
+                lr_gate_step(m, r[REC - 4], r[REC - 2], fade, write);
+                vv *= write;
+            }
+            const float o = lr_walk_token<R, LANES, RULE>(S, r + DP, r, r + 2 * DP, fade, vv, r[REC - 4], r[REC - 3], sub);
+            if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt), h, col, o, m);
         }
         __syncthreads();                                                   // this chunk's buffer may be filled again
     }
+    if (smax && sub == 0) *smax = m;
     if (srow) {
 #pragma unroll
         for (int i = 0; i < R / 4; ++i)
@@ -427,7 +497,7 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
 template <typename T, int R, int LANES, int COLS, int RULE>
 static int launch_linear_state_ready(const LinearStateArgs& p, float* work, int n_tokens, cudaStream_t stream) {
     constexpr int REC = LrRecord<RULE, LANES * R>::SIZE;
-    const int tiles = (p.vdim + COLS - 1) / COLS, vp = tiles * COLS;
+    const int tiles = (LR_COLUMNS(RULE, p.vdim) + COLS - 1) / COLS, vp = tiles * COLS;
     const long long pairs = (long long)n_tokens * p.heads;
     float* rec = work;
     float* pv = work + (size_t)pairs * REC;
@@ -451,7 +521,7 @@ static int launch_linear_state_ready(const LinearStateArgs& p, float* work, int 
 static long long linear_state_work_floats(int rule, int n_tokens, int heads, int dim, int vdim) {
     const int dp = dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256;
     const int cols = LR_COLS;
-    const int rec = (LR_PER_ENTRY(rule) ? 3 : 2) * dp + 4, vp = (vdim + cols - 1) / cols * cols;
+    const int rec = (LR_PER_ENTRY(rule) ? 3 : 2) * dp + 4, vp = (LR_COLUMNS(rule, vdim) + cols - 1) / cols * cols;
     return (long long)n_tokens * heads * (rec + vp);
 }
 
@@ -479,15 +549,18 @@ ZI_EXPORT int zi_linear_state(int rule, const void* q, long long ldq, const void
                               const void* a, long long lda, const void* b, long long ldb, int dtype, const float* dt_bias,
                               const float* a_log, const float* decay, float* state, long long slot_stride, const int* slots,
                               const int* bounds, float* y, int n_tokens, int n_segments, int heads, int kv_heads, int dim, int vdim,
-                              int act_silu, int decay_per_head, float q_scale, float unit_eps, float* work, long long work_floats, cudaStream_t stream) {
+                              int act_silu, int decay_per_head, float q_scale, float unit_eps, float* den, float gate_cap, float* work,
+                              long long work_floats, cudaStream_t stream) {
     if (n_tokens <= 0 || n_segments <= 0) return 0;
-    if (rule < 0 || rule > 2) return zi_fail("linear_state: rule %d is none of 0 (delta), 1 (decay), 2 (forget)", rule);
+    if (rule < 0 || rule > 3) return zi_fail("linear_state: rule %d is none of 0 (delta), 1 (decay), 2 (forget), 3 (expgate)", rule);
     if (heads <= 0 || kv_heads <= 0 || heads % kv_heads) return zi_fail("linear_state: %d heads cannot share %d query/key heads", heads, kv_heads);
     if (dim <= 0 || dim > 256 || vdim <= 0) return zi_fail("linear_state: dim=%d must lie in 1 .. 256 and vdim=%d be positive", dim, vdim);
     if (heads > 65535) return zi_fail("linear_state: too many heads: %d", heads);
     if (rule == 0 && (!a || !b || !dt_bias || !a_log)) return zi_fail("linear_state: the delta rule needs a, b, dt_bias and A_log");
     if (rule == 1 && !decay) return zi_fail("linear_state: the decay rule needs the heads' decays");
     if (rule == 2 && (!a || !dt_bias || heads != kv_heads)) return zi_fail("linear_state: the forget rule needs the gates, their lower bounds and a query head per head");
+    if (rule == 3 && (!a || !b || !dt_bias || !a_log || !den || !(gate_cap > 0.0f)))
+        return zi_fail("linear_state: the expgate rule needs both gates' projections and biases, a positive cap and room for the divisors");
     if (!bounds && n_segments != n_tokens) return zi_fail("linear_state: without bounds every segment is one token");
     LinearStateArgs p;
     p.q = q; p.k = k; p.v = v; p.a = a; p.b = b;
@@ -495,7 +568,7 @@ ZI_EXPORT int zi_linear_state(int rule, const void* q, long long ldq, const void
     p.dt_bias = dt_bias; p.a_log = a_log; p.decay = decay;
     p.state = state; p.slot_stride = slot_stride; p.slots = slots; p.bounds = bounds; p.y = y;
     p.n_segments = n_segments; p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.act_silu = act_silu; p.decay_per_head = decay_per_head;
-    p.q_scale = q_scale; p.unit_eps = unit_eps;
+    p.q_scale = q_scale; p.unit_eps = unit_eps; p.den = den; p.gate_cap = gate_cap;
     if (work) {
         // inputs made ready first, then the walk
         if (((size_t)work & 15) != 0) return zi_fail("linear_state: the workspace must start on a 16-byte boundary");
@@ -504,6 +577,7 @@ ZI_EXPORT int zi_linear_state(int rule, const void* q, long long ldq, const void
         ZI_DISPATCH(dtype, T, {
             if (rule == LR_DELTA) return pick_linear_state_ready<T, LR_DELTA>(p, work, n_tokens, stream);
             if (rule == LR_FORGET) return pick_linear_state_ready<T, LR_FORGET>(p, work, n_tokens, stream);
+            if (rule == LR_EXPGATE) return pick_linear_state_ready<T, LR_EXPGATE>(p, work, n_tokens, stream);
             return pick_linear_state_ready<T, LR_DECAY>(p, work, n_tokens, stream);
         });
         return 0;
@@ -511,6 +585,7 @@ ZI_EXPORT int zi_linear_state(int rule, const void* q, long long ldq, const void
     ZI_DISPATCH(dtype, T, {
         if (rule == LR_DELTA) return pick_linear_state<T, LR_DELTA>(p, stream);
         if (rule == LR_FORGET) return pick_linear_state<T, LR_FORGET>(p, stream);
+        if (rule == LR_EXPGATE) return pick_linear_state<T, LR_EXPGATE>(p, stream);
         return pick_linear_state<T, LR_DECAY>(p, stream);
     });
     return 0;
@@ -518,7 +593,7 @@ ZI_EXPORT int zi_linear_state(int rule, const void* q, long long ldq, const void
 
 // ---------------------------------------------------------------------------------------
 // out[n, c] = y[n, c] / sqrt(mean_group(y^2) + eps) * w[c mod w_len] * gate(z[n, c]), gate 0: sigmoid, 1: SiLU, 2: none (z unused); the mean over each of n_groups
-// equal parts of a row.  y float32; z (rows may be strided) and out of the step's type.  One block per row; a group's sum
+// equal parts of a row.  den (optional, [n, n_groups]): y stands for y / den[n, group].  y float32; z (rows may be strided) and out of the step's type.  One block per row; a group's sum
 // is taken by one warp when there are at least as many groups as warps, else by the whole block, group after group.
 // ---------------------------------------------------------------------------------------
 #define GN_THREADS 256
@@ -531,7 +606,7 @@ __device__ __forceinline__ float gn_gate(const T* zr, int c, int gate) {
 
 template <typename T, typename TW>
 __global__ void __launch_bounds__(GN_THREADS)
-group_rmsnorm_gate_kernel(const float* __restrict__ y, const T* __restrict__ z, long long ldz, const TW* __restrict__ w, int w_len,
+group_rmsnorm_gate_kernel(const float* __restrict__ y, const float* __restrict__ den, const T* __restrict__ z, long long ldz, const TW* __restrict__ w, int w_len,
                           T* __restrict__ out, int inner, int n_groups, float eps, int gate) {
     __shared__ float scratch[32];
     const int n = blockIdx.x, gw = inner / n_groups;
@@ -541,37 +616,39 @@ group_rmsnorm_gate_kernel(const float* __restrict__ y, const T* __restrict__ z, 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (n_groups >= GN_THREADS / 32) {
         for (int g = warp; g < n_groups; g += GN_THREADS / 32) {
+            const float dv = den ? 1.0f / den[(size_t)n * n_groups + g] : 1.0f;
             float ss = 0.0f;
-            for (int j = lane; j < gw; j += 32) { const float x = yr[g * gw + j]; ss = fmaf(x, x, ss); }
+            for (int j = lane; j < gw; j += 32) { const float x = yr[g * gw + j] * dv; ss = fmaf(x, x, ss); }
             ss = warp_sum(ss);
             const float r = 1.0f / sqrtf(ss / (float)gw + eps);
             for (int j = lane; j < gw; j += 32) {
                 const int c = g * gw + j;
-                orow[c] = from_f32<T>(yr[c] * r * to_f32<TW>(w[c % w_len]) * gn_gate<T>(zr, c, gate));
+                orow[c] = from_f32<T>(yr[c] * dv * r * to_f32<TW>(w[c % w_len]) * gn_gate<T>(zr, c, gate));
             }
         }
         return;
     }
     for (int g = 0; g < n_groups; ++g) {
+        const float dv = den ? 1.0f / den[(size_t)n * n_groups + g] : 1.0f;
         float ss = 0.0f;
-        for (int j = threadIdx.x; j < gw; j += GN_THREADS) { const float x = yr[g * gw + j]; ss = fmaf(x, x, ss); }
+        for (int j = threadIdx.x; j < gw; j += GN_THREADS) { const float x = yr[g * gw + j] * dv; ss = fmaf(x, x, ss); }
         ss = block_sum(ss, scratch);
         const float r = 1.0f / sqrtf(ss / (float)gw + eps);
         for (int j = threadIdx.x; j < gw; j += GN_THREADS) {
             const int c = g * gw + j;
-            orow[c] = from_f32<T>(yr[c] * r * to_f32<TW>(w[c % w_len]) * gn_gate<T>(zr, c, gate));
+            orow[c] = from_f32<T>(yr[c] * dv * r * to_f32<TW>(w[c % w_len]) * gn_gate<T>(zr, c, gate));
         }
     }
 }
 
-ZI_EXPORT int zi_group_rmsnorm_gate(const float* y, const void* z, int dtype, long long ldz, const void* w, int w_dtype, int w_len,
+ZI_EXPORT int zi_group_rmsnorm_gate(const float* y, const float* den, const void* z, int dtype, long long ldz, const void* w, int w_dtype, int w_len,
                                     void* out, int n_tokens, int inner, int n_groups, float eps, int gate, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (inner <= 0 || n_groups <= 0 || inner % n_groups) return zi_fail("group_rmsnorm_gate: %d groups do not divide %d", n_groups, inner);
     if (gate < 0 || gate > 2 || (gate != 2 && !z)) return zi_fail("group_rmsnorm_gate: gate %d is none of 0 (sigmoid), 1 (SiLU), 2 (none), or its input is missing", gate);
     if (w_len <= 0 || inner % w_len) return zi_fail("group_rmsnorm_gate: a weight of %d entries does not tile a row of %d", w_len, inner);
     ZI_DISPATCH(dtype, T, ZI_DISPATCH(w_dtype, TW, {
-        group_rmsnorm_gate_kernel<T, TW><<<n_tokens, GN_THREADS, 0, stream>>>(y, (const T*)z, ldz, (const TW*)w, w_len, (T*)out, inner,
+        group_rmsnorm_gate_kernel<T, TW><<<n_tokens, GN_THREADS, 0, stream>>>(y, den, (const T*)z, ldz, (const TW*)w, w_len, (T*)out, inner,
                                                                             n_groups, eps, gate);
     }););
     return zi_check_launch("group_rmsnorm_gate");

@@ -149,6 +149,41 @@ ZI_EXPORT int zi_gated_clamp_mul(const void* gate_up, void* out, int dtype, int 
 }
 
 // ---------------------------------------------------------------------------------------
+// Gated GELU.  x [rows, 2 * inter]: out[n, j] = gelu_tanh(x[n, j]) * x[n, inter + j]
+// ---------------------------------------------------------------------------------------
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+gated_gelu_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int inter, size_t units) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < units; i += (size_t)gridDim.x * blockDim.x) {
+        if (VEC) {
+            const size_t per = inter / 8, n = i / per, j = (i - n * per) * 8;
+            float g[8], u[8];
+            load8(x + n * 2 * inter + j, g);
+            load8(x + n * 2 * inter + inter + j, u);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) g[e] = gelu_tanh(g[e]) * u[e];
+            store8(out + n * inter + j, g);
+        } else {
+            const size_t n = i / inter, j = i - n * inter;
+            out[i] = from_f32<T>(gelu_tanh(to_f32<T>(x[n * 2 * inter + j])) * to_f32<T>(x[n * 2 * inter + inter + j]));
+        }
+    }
+}
+
+ZI_EXPORT int zi_gated_gelu_mul(const void* gate_up, void* out, int dtype, int rows, int inter, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (inter <= 0) return zi_fail("gated_gelu_mul: width %d must be positive", inter);
+    const bool vec = inter % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 31) == 0;
+    const size_t units = (size_t)rows * inter / (vec ? 8 : 1), want = (units + 255) / 256;
+    const int blocks = (int)(want > 148 * 32 ? 148 * 32 : want);
+    ZI_DISPATCH(dtype, T, {
+        if (vec) gated_gelu_mul_kernel<T, true><<<blocks, 256, 0, stream>>>((const T*)gate_up, (T*)out, inter, units);
+        else gated_gelu_mul_kernel<T, false><<<blocks, 256, 0, stream>>>((const T*)gate_up, (T*)out, inter, units);
+    });
+    return zi_check_launch("gated_gelu_mul");
+}
+
+// ---------------------------------------------------------------------------------------
 // RMSNorm of `width` columns of each row of x, written into the pages of a paged cache with one
 // plane and one head per token (a latent):  y = (w * x) * rstd,  rstd = 1/sqrt(mean(x^2) + eps).
 //   x      [n_tokens, row_stride]; the first `width` columns of a row are normed
@@ -481,9 +516,31 @@ __global__ void sigmoid_mul_kernel(T* __restrict__ a, const T* __restrict__ g, l
     }
 }
 
+// The same with eight entries per access; width and ldg multiples of 8, pointers aligned for it.  The same bits.
+template <typename T>
+__global__ void __launch_bounds__(128)
+sigmoid_mul_vec8_kernel(T* __restrict__ a, const T* __restrict__ g, long long ldg, int width8, size_t total8) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total8; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t n = i / width8;
+        const int j = (int)(i - n * width8) * 8;
+        float av[8], gv[8];
+        load8(a + i * 8, av); load8(g + n * ldg + j, gv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) av[e] = av[e] / (1.0f + expf(-gv[e]));
+        store8(a + i * 8, av);
+    }
+}
+
 ZI_EXPORT int zi_sigmoid_mul(void* a, const void* g, int dtype, long long ldg, int rows, int width, cudaStream_t stream) {
     if (rows <= 0 || width <= 0) return 0;
     const size_t total = (size_t)rows * width;
+    if (width % 8 == 0 && ldg % 8 == 0 && (((uintptr_t)a | (uintptr_t)g) & (dtype == ZI_BF16 ? 15 : 31)) == 0) {
+        const size_t total8 = total / 8, blocks = (total8 + 127) / 128;
+        ZI_DISPATCH(dtype, T, {
+            sigmoid_mul_vec8_kernel<T><<<(int)(blocks > 148 * 32 ? 148 * 32 : blocks), 128, 0, stream>>>((T*)a, (const T*)g, ldg, width / 8, total8);
+        });
+        return zi_check_launch("sigmoid_mul");
+    }
     const size_t want = (total + 255) / 256;
     ZI_DISPATCH(dtype, T, {
         sigmoid_mul_kernel<T><<<(int)(want > 148 * 16 ? 148 * 16 : want), 256, 0, stream>>>((T*)a, (const T*)g, ldg, width, total);
@@ -682,8 +739,7 @@ __global__ void gelu_mul_rows_kernel(const T* __restrict__ t, long long ldt, con
         const int j = (int)(i - n * width);
         int id = ids[n];
         id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
-        const float z = to_f32<T>(t[n * ldt + j]);
-        const float g = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+        const float g = gelu_tanh(to_f32<T>(t[n * ldt + j]));
         out[i] = from_f32<T>(g * to_f32<TT>(table[(size_t)id * ld_table + col0 + j]));
     }
 }
@@ -1056,4 +1112,344 @@ ZI_EXPORT int zi_row_gate(const void* x, int dtype, long long ldx, const void* w
         else row_gate_kernel<T, TW, false><<<blocks, RG_WARPS * 32, 0, stream>>>((const T*)x, ldx, (const TW*)w, g, rows, K);
     }););
     return zi_check_launch("row_gate");
+}
+
+// ---------------------------------------------------------------------------------------
+// Normed queries and keys: what a layer's q | k | v product needs before attention, in one kernel.
+//   x        [n_tokens, ldx]: n_q query heads and n_k key heads of qk_dim entries, then n_k value heads of v_dim entries
+//   norm     0: none;  1: every query and key head u becomes u / sqrt(mean(u^2) + eps) * w, qw and kw [qk_dim] shared by the heads;
+//            2: the same over all query heads of a token at once (qw [n_q * qk_dim]) and over all its key heads (kw [n_k * qk_dim])
+//   turn     then the first rot_dims entries of every query and key head turn by position (pairing as in rotary_kernel)
+//   heat     then queries are multiplied by 1 + heat_coef ln(floor((pos + 1) / heat_every) + 1)      (heat_every 0: not)
+//   mix      values become (1 - lambda) v + lambda v_first[n, :]                                     (v_first null: not)
+//   q_out    [n_tokens, n_q * row_dim];  cache: keys and values appended, rows row_dim wide, zero past a head's own entries
+// One block per token.  The token's queries and keys pass through shared memory as float32; a sum of squares has one order
+// that depends on the sizes alone.  VEC: eight entries per access.
+// ---------------------------------------------------------------------------------------
+#define QP_THREADS 256
+struct QkPrepArgs {
+    const float* qw; const float* kw; const float* inv_freq;
+    int n_q, n_k, qk_dim, v_dim, row_dim, norm, rot_dims, interleaved, page_size, max_blocks;
+    long long page_stride, kv_stride, ldx, ld_first;
+    float eps, mag, heat_coef, heat_every, lambda;
+};
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(QP_THREADS)
+qk_norm_append_kernel(const T* __restrict__ x, T* __restrict__ q_out, T* __restrict__ cache, const T* __restrict__ v_first,
+                      const int* __restrict__ tables, const int* __restrict__ tok_seg, const int* __restrict__ pos, const QkPrepArgs a) {
+    extern __shared__ float qp_smem[];                 // the rows of q and k | cos, sin | a factor per head
+    __shared__ float scratch[96];
+    const int n = blockIdx.x, half = a.rot_dims >> 1, heads = a.n_q + a.n_k;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int q_len = a.n_q * a.qk_dim, qk_len = heads * a.qk_dim;
+    float* row = qp_smem;
+    float* cs = row + (qk_len + 3) / 4 * 4;
+    float* factor = cs + a.rot_dims;
+    const int p = pos[n];
+    const int seg = tok_seg ? tok_seg[n] : n;
+    const int page = tables[(size_t)seg * a.max_blocks + p / a.page_size];
+    T* page_base = cache + (size_t)page * a.page_stride + (size_t)(p % a.page_size) * a.row_dim;
+    const T* xr = x + (size_t)n * a.ldx;
+    // values need nothing of the rest
+    const T* vr = xr + qk_len;
+    const T* fr = v_first ? v_first + (size_t)n * a.ld_first : nullptr;
+    if (VEC) {
+        const int per = a.row_dim >> 3;
+        for (int idx = threadIdx.x; idx < a.n_k * per; idx += QP_THREADS) {
+            const int g = idx / per, d = (idx - g * per) * 8;
+            float v[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+            if (d < a.v_dim) {
+                load8(vr + g * a.v_dim + d, v);
+                if (fr) {
+                    float f[8];
+                    load8(fr + g * a.v_dim + d, f);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) v[e] = (1.0f - a.lambda) * v[e] + a.lambda * f[e];
+                }
+            }
+            store8(page_base + a.kv_stride + (size_t)g * a.page_size * a.row_dim + d, v);
+        }
+    } else {
+        for (int idx = threadIdx.x; idx < a.n_k * a.row_dim; idx += QP_THREADS) {
+            const int g = idx / a.row_dim, d = idx - g * a.row_dim;
+            float v = 0.0f;
+            if (d < a.v_dim) {
+                v = to_f32<T>(vr[g * a.v_dim + d]);
+                if (fr) v = (1.0f - a.lambda) * v + a.lambda * to_f32<T>(fr[g * a.v_dim + d]);
+            }
+            page_base[a.kv_stride + (size_t)g * a.page_size * a.row_dim + d] = from_f32<T>(v);
+        }
+    }
+    for (int i = threadIdx.x; i < half; i += QP_THREADS) {
+        float s, c;
+        sincosf((float)p * a.inv_freq[i], &s, &c);
+        cs[i] = c * a.mag;
+        cs[half + i] = s * a.mag;
+    }
+    const float heat = a.heat_every > 0.0f ? fmaf(a.heat_coef, logf(floorf((float)(p + 1) / a.heat_every) + 1.0f), 1.0f) : 1.0f;
+    float sq = 0.0f, sk = 0.0f, unused = 0.0f;
+    if (VEC) {
+        for (int j = threadIdx.x * 8; j < qk_len; j += QP_THREADS * 8) {
+            float v[8], s = 0.0f;
+            load8(xr + j, v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+            store8(row + j, v);
+            if (j < q_len) sq += s; else sk += s;      // a group of eight lies in one head
+        }
+    } else {
+        for (int j = threadIdx.x; j < qk_len; j += QP_THREADS) {
+            const float v = to_f32<T>(xr[j]);
+            row[j] = v;
+            if (j < q_len) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
+        }
+    }
+    if (a.norm == 2) {
+        block_sum3(sq, sk, unused, scratch);
+        const float rq = 1.0f / sqrtf(sq / (float)q_len + a.eps), rk = 1.0f / sqrtf(sk / (float)(qk_len - q_len) + a.eps);
+        for (int h = threadIdx.x; h < heads; h += QP_THREADS) factor[h] = h < a.n_q ? rq : rk;
+    } else {
+        __syncthreads();
+        for (int h = warp; h < heads; h += QP_THREADS / 32) {
+            float ss = 0.0f;
+            if (a.norm == 1) {
+                for (int d = lane; d < a.qk_dim; d += 32) ss = fmaf(row[h * a.qk_dim + d], row[h * a.qk_dim + d], ss);
+                ss = warp_sum(ss);
+            }
+            if (lane == 0) factor[h] = a.norm == 1 ? 1.0f / sqrtf(ss / (float)a.qk_dim + a.eps) : 1.0f;
+        }
+    }
+    __syncthreads();
+    // write: eight entries of a head per thread; rows of the cache and heads of q_out are multiples of 8 entries
+    const int per = a.row_dim >> 3;
+    for (int idx = threadIdx.x; idx < heads * per; idx += QP_THREADS) {
+        const int h = idx / per, d0 = (idx - h * per) * 8;
+        const float* hr = row + h * a.qk_dim;
+        const float* w = a.norm == 0 ? nullptr : (h < a.n_q ? a.qw + (a.norm == 2 ? h * a.qk_dim : 0) : a.kw + (a.norm == 2 ? (h - a.n_q) * a.qk_dim : 0));
+        const float r = factor[h], last = h < a.n_q ? heat : 1.0f;
+        auto normed = [&](int d) { return w ? hr[d] * r * w[d] : hr[d]; };
+        float o[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            const int d = d0 + e;
+            float v = 0.0f;
+            if (d < a.rot_dims) {
+                const int i = a.interleaved ? d >> 1 : (d < half ? d : d - half);
+                const int lo_at = a.interleaved ? d & ~1 : i, hi_at = a.interleaved ? d | 1 : i + half;
+                float olo, ohi;
+                rotate_pair(normed(lo_at), normed(hi_at), cs[i], cs[half + i], &olo, &ohi);
+                v = d == lo_at ? olo : ohi;
+            } else if (d < a.qk_dim) {
+                v = normed(d);
+            }
+            o[e] = v * last;
+        }
+        T* dst = h < a.n_q ? q_out + ((size_t)n * a.n_q + h) * a.row_dim : page_base + (size_t)(h - a.n_q) * a.page_size * a.row_dim;
+        store8(dst + d0, o);
+    }
+}
+
+ZI_EXPORT int zi_qk_norm_append(const void* x, int dtype, long long ldx, void* q_out, void* cache, const int* tables, const int* tok_seg,
+                                const int* pos, const float* qw, const float* kw, int norm, float eps, const float* inv_freq, float mag,
+                                int rot_dims, int interleaved, float heat_coef, float heat_every, const void* v_first, long long ld_first,
+                                float lambda, int n_tokens, int n_q, int n_k, int qk_dim, int v_dim, int row_dim, int page_size, int max_blocks,
+                                long long page_stride, long long kv_stride, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_q <= 0 || n_k <= 0 || qk_dim <= 0 || v_dim <= 0) return zi_fail("qk_norm_append: heads %d / %d of %d and %d entries", n_q, n_k, qk_dim, v_dim);
+    if (rot_dims < 0 || (rot_dims & 1) || rot_dims > qk_dim) return zi_fail("qk_norm_append: a span of %d entries does not fit a head of %d (or is odd)", rot_dims, qk_dim);
+    if (row_dim % 8 || row_dim < qk_dim || row_dim < v_dim) return zi_fail("qk_norm_append: rows of %d entries cannot hold heads of %d and %d", row_dim, qk_dim, v_dim);
+    if (norm < 0 || norm > 2 || (norm && (!qw || !kw))) return zi_fail("qk_norm_append: norm %d is none of 0, 1, 2, or its weights are missing", norm);
+    if (!cache || !tables || page_size <= 0 || max_blocks <= 0 || kv_stride == 0) return zi_fail("qk_norm_append: the cache append needs tables, a page size and two planes");
+    if (rot_dims > 0 && !inv_freq) return zi_fail("qk_norm_append: a turned span needs its frequencies");
+    const size_t align = dtype == ZI_BF16 ? 15 : 31;
+    if ((((uintptr_t)q_out | (uintptr_t)cache) & align) || page_stride % 8 || kv_stride % 8) return zi_fail("qk_norm_append: q_out and cache must be aligned for eight entries");
+    const bool vec = qk_dim % 8 == 0 && v_dim % 8 == 0 && ldx % 8 == 0 && ((uintptr_t)x & align) == 0 &&
+                     (!v_first || (ld_first % 8 == 0 && ((uintptr_t)v_first & align) == 0));
+    const size_t smem = ((size_t)((n_q + n_k) * qk_dim + 3) / 4 * 4 + rot_dims + n_q + n_k) * sizeof(float);
+    if (smem > 200 * 1024) return zi_fail("qk_norm_append: %d + %d heads of %d entries are too many for one block", n_q, n_k, qk_dim);
+    const QkPrepArgs a{qw, kw, inv_freq, n_q, n_k, qk_dim, v_dim, row_dim, norm, rot_dims, interleaved, page_size, max_blocks,
+                       page_stride, kv_stride, ldx, ld_first, eps, mag, heat_coef, heat_every, lambda};
+    ZI_DISPATCH(dtype, T, {
+        auto kernel = vec ? qk_norm_append_kernel<T, true> : qk_norm_append_kernel<T, false>;
+        if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+            return zi_fail("qk_norm_append: cannot reserve %zu bytes of shared memory", smem);
+        kernel<<<n_tokens, QP_THREADS, smem, stream>>>((const T*)x, (T*)q_out, (T*)cache, (const T*)v_first, tables, tok_seg, pos, a);
+    });
+    return zi_check_launch("qk_norm_append");
+}
+
+// ---------------------------------------------------------------------------------------
+// Branches that read the same normed input join the float32 residual stream together, and the next norm follows:
+//     v = h[row] + s,   s = y + f,  or with a second output y2 that is joined with y:  s = (U(y) w1 + U(y2) w2) / 2 + f
+//     h[row] = v        where write_h is set
+//     out[r] = v / sqrt(mean(v^2) + eps) * w
+// with U(u) = u / sqrt(mean(u^2) + join_eps) over the row.  Each of y, y2, f may be absent (null) or come as `parts` float32 sums
+// (yp, fp >= 1: part k is k * part_stride entries further on), which are added in order and rounded to the step's type.
+// row = row_idx[r] where row_idx is given (then h is not written), else r.  h float32; y, y2, f, out of the step's type; w1, w2,
+// w float32.  One block per row; C > 0: eight entries per access and C such groups per thread (hidden <= 2048 C), everything a
+// thread needs asked for before the sums are taken; C = 0: entry by entry through shared memory.
+// ---------------------------------------------------------------------------------------
+struct FoldArgs {
+    float* h; const void* y; const void* y2; const void* f; const float* w1; const float* w2; const float* w; const int* row_idx;
+    int yp, fp, write_h, hidden;
+    long long part_stride;
+    float join_eps, eps;
+};
+
+template <typename T>
+__device__ __forceinline__ void fold_load8(const void* src, int parts, long long stride, size_t at, float (&v)[8]) {
+    if (parts == 0) { load8((const T*)src + at, v); return; }
+    load8((const float*)src + at, v);
+    for (int k = 1; k < parts; ++k) {
+        float t[8];
+        load8((const float*)src + (size_t)k * stride + at, t);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] += t[e];
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = to_f32<T>(from_f32<T>(v[e]));
+}
+template <typename T>
+__device__ __forceinline__ float fold_load1(const void* src, int parts, long long stride, size_t at) {
+    if (parts == 0) return to_f32<T>(((const T*)src)[at]);
+    float v = ((const float*)src)[at];
+    for (int k = 1; k < parts; ++k) v += ((const float*)src)[(size_t)k * stride + at];
+    return to_f32<T>(from_f32<T>(v));
+}
+
+template <typename T, int C>
+__global__ void __launch_bounds__(256)
+branches_rmsnorm_kernel(const FoldArgs a, T* __restrict__ out) {
+    __shared__ float scratch[96];
+    const size_t r = blockIdx.x, row = a.row_idx ? (size_t)a.row_idx[r] : r, base = row * a.hidden;
+    const int hidden = a.hidden;
+    const float inv_n = 1.0f / (float)hidden;
+    if constexpr (C > 0) {
+        float v[C][8], y[C][8], y2[C][8], w[C][8], w1[C][8], w2[C][8];
+        float s1 = 0.0f, s2 = 0.0f, unused = 0.0f;
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            const int j = (c * 256 + threadIdx.x) * 8;
+            if (j < hidden) {
+                load8(a.h + base + j, v[c]);
+                if (a.w) load8(a.w + j, w[c]);
+                if (a.y) {
+                    fold_load8<T>(a.y, a.yp, a.part_stride, base + j, y[c]);
+                    if (a.y2) {
+                        load8((const T*)a.y2 + base + j, y2[c]);
+                        load8(a.w1 + j, w1[c]);
+                        load8(a.w2 + j, w2[c]);
+                    }
+                }
+                if (a.f) {
+                    float f[8];
+                    fold_load8<T>(a.f, a.fp, a.part_stride, base + j, f);
+                    // a branch that is not joined is added to the other first: their sum joins the stream
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) {
+                        if (a.y && !a.y2) y[c][e] += f[e];
+                        else v[c][e] += f[e];
+                    }
+                }
+                if (a.y2) {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) { s1 = fmaf(y[c][e], y[c][e], s1); s2 = fmaf(y2[c][e], y2[c][e], s2); }
+                }
+            }
+        }
+        float r1 = 0.0f, r2 = 0.0f;
+        if (a.y2) {
+            block_sum3(s1, s2, unused, scratch);
+            r1 = 0.5f / sqrtf(s1 * inv_n + a.join_eps);
+            r2 = 0.5f / sqrtf(s2 * inv_n + a.join_eps);
+        }
+        float ss = 0.0f;
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            const int j = (c * 256 + threadIdx.x) * 8;
+            if (j < hidden) {
+                if (a.y) {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e)
+                        v[c][e] += a.y2 ? y[c][e] * r1 * w1[c][e] + y2[c][e] * r2 * w2[c][e] : y[c][e];
+                }
+                if (a.write_h) store8(a.h + base + j, v[c]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss = fmaf(v[c][e], v[c][e], ss);
+            }
+        }
+        if (!out) return;
+        __syncthreads();
+        ss = block_sum(ss, scratch);
+        const float rr = 1.0f / sqrtf(ss * inv_n + a.eps);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            const int j = (c * 256 + threadIdx.x) * 8;
+            if (j < hidden) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[c][e] = v[c][e] * rr * w[c][e];
+                store8(out + r * hidden + j, v[c]);
+            }
+        }
+    } else {
+        extern __shared__ float fold_row[];
+        float r1 = 0.0f, r2 = 0.0f;
+        if (a.y2) {
+            float s1 = 0.0f, s2 = 0.0f, unused = 0.0f;
+            for (int j = threadIdx.x; j < hidden; j += 256) {
+                const float p = fold_load1<T>(a.y, a.yp, a.part_stride, base + j), q = to_f32<T>(((const T*)a.y2)[base + j]);
+                s1 = fmaf(p, p, s1);
+                s2 = fmaf(q, q, s2);
+            }
+            block_sum3(s1, s2, unused, scratch);
+            r1 = 0.5f / sqrtf(s1 * inv_n + a.join_eps);
+            r2 = 0.5f / sqrtf(s2 * inv_n + a.join_eps);
+        }
+        float ss = 0.0f;
+        for (int j = threadIdx.x; j < hidden; j += 256) {
+            float v = a.h[base + j];
+            const float f = a.f ? fold_load1<T>(a.f, a.fp, a.part_stride, base + j) : 0.0f;
+            if (a.y) {
+                const float p = fold_load1<T>(a.y, a.yp, a.part_stride, base + j);
+                if (a.y2) v = (v + f) + (p * r1 * a.w1[j] + to_f32<T>(((const T*)a.y2)[base + j]) * r2 * a.w2[j]);
+                else v += p + f;
+            } else {
+                v += f;
+            }
+            if (a.write_h) a.h[base + j] = v;
+            fold_row[j] = v;
+            ss = fmaf(v, v, ss);
+        }
+        if (!out) return;
+        __syncthreads();
+        ss = block_sum(ss, scratch);
+        const float rr = 1.0f / sqrtf(ss * inv_n + a.eps);
+        for (int j = threadIdx.x; j < hidden; j += 256) out[r * hidden + j] = from_f32<T>(fold_row[j] * rr * a.w[j]);
+    }
+}
+
+ZI_EXPORT int zi_branches_rmsnorm(float* h, const void* y, int y_parts, const void* y2, const void* f, int f_parts, long long part_stride,
+                                  int dtype, const float* w1, const float* w2, float join_eps, const float* w, float eps, void* out,
+                                  const int* row_idx, int rows, int hidden, int write_h, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (hidden <= 0) return zi_fail("branches_rmsnorm: hidden=%d", hidden);
+    if (y2 && (!y || !w1 || !w2)) return zi_fail("branches_rmsnorm: two joined branches need both outputs and their weights");
+    if (out && !w) return zi_fail("branches_rmsnorm: an output needs its norm's weight");
+    if (row_idx && write_h) return zi_fail("branches_rmsnorm: chosen rows leave the stream as it is");
+    const FoldArgs a{h, y, y2, f, w1, w2, w, row_idx, y_parts, f_parts, write_h, hidden, part_stride, join_eps, eps};
+    // which form runs depends on the sizes and on where the buffers start, never on the rows of the step
+    const bool vec = hidden % 8 == 0 && hidden <= 8192 && part_stride % 8 == 0 &&
+                     (((size_t)h | (size_t)y | (size_t)y2 | (size_t)f | (size_t)out | (size_t)w1 | (size_t)w2 | (size_t)w) & 15) == 0;
+    ZI_DISPATCH(dtype, T, {
+        if (vec && hidden <= 2048) branches_rmsnorm_kernel<T, 1><<<rows, 256, 0, stream>>>(a, (T*)out);
+        else if (vec && hidden <= 4096) branches_rmsnorm_kernel<T, 2><<<rows, 256, 0, stream>>>(a, (T*)out);
+        else if (vec) branches_rmsnorm_kernel<T, 4><<<rows, 256, 0, stream>>>(a, (T*)out);
+        else {
+            const size_t smem = (size_t)hidden * sizeof(float);
+            if (smem > 48 * 1024) return zi_fail("branches_rmsnorm: hidden=%d is not supported", hidden);
+            branches_rmsnorm_kernel<T, 0><<<rows, 256, smem, stream>>>(a, (T*)out);
+        }
+    });
+    return zi_check_launch("branches_rmsnorm");
 }

@@ -211,3 +211,26 @@ static inline cudaError_t zi_launch(void (*kernel)(KArgs...), dim3 grid, dim3 bl
         else if ((code) == ZI_BF16) { typedef bf16 T; __VA_ARGS__ }   \
         else return zi_fail("unknown dtype code %d", (int)(code));    \
     } while (0)
+
+// ---- the tanh form of GELU -----------------------------------------------------------------
+#define GELU_TANH_SLOPE 0.7978845608028654f     // sqrt(2 / pi)
+#define GELU_TANH_CUBIC 0.044715f
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.0f + tanhf(GELU_TANH_SLOPE * (z + GELU_TANH_CUBIC * z * z * z)));
+}
+
+// ---- which keys a query sees -----------------------------------------------------------
+// The first key that the query at position P may see.  window > 0: the last `window` keys, the query's own included; window
+// < 0: the keys of the query's own chunk of -window positions, chunks counted from position 0; 0: every key.  Grows with P.
+__device__ __forceinline__ int first_visible_key(int P, int window) {
+    if (window > 0) return P - window + 1 > 0 ? P - window + 1 : 0;
+    if (window < 0 && P > 0) return P - P % -window;
+    return 0;
+}
+
+// A number per query head and distance that joins a score (after the scale and the cap): table [n_heads, len], float32;
+// distances of len - 1 and more share the last entry.  table null: none.
+struct DistanceBias {
+    const float* table;
+    int len;
+};

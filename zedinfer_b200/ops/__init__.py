@@ -39,7 +39,7 @@ __all__ = ["KernelError", "embedding", "rmsnorm", "add_rmsnorm", "rope_append", 
            "moe_gather_rows", "gemm_tcgen05_grouped", "route", "rotary", "latent_prepare", "sigmoid_mul", "segment_bounds",
            "causal_conv_silu", "conv_state_update", "ssm_scan", "gated_group_rmsnorm", "rotary_norm", "norm_add", "gelu_mul_rows",
            "linear_state", "linear_state_work_floats", "group_rmsnorm_gate", "tanh_norm", "tanh_norm_fold", "rms_pair_mean", "poly_norm",
-           "row_gate"]
+           "row_gate", "linear_gelu_mul", "gated_gelu_mul", "linear_state_floats", "qk_norm_append", "branches_rmsnorm"]
 
 
 def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
@@ -258,13 +258,14 @@ def _small_m_ok(x: torch.Tensor, w: torch.Tensor, fused: Optional[str] = None) -
 
 
 def gemm_smallm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-                silu_mul: bool = False, gated: Optional[tuple] = None, relu2: bool = False) -> None:
+                silu_mul: bool = False, gated: Optional[tuple] = None, relu2: bool = False, gelu_mul: bool = False) -> None:
     """``out = x @ w.T + bias`` for at most 16 rows of ``x``: weights stream once from memory into the
     tensor cores.  ``silu_mul``: ``w`` is ``[2*I, K]`` (gate rows, then up rows) and ``out[m, j] =
     up * gate / (1 + exp(-gate))``.  ``gated = (limit, slope, up_offset)``: the same stacked weight with the clamped,
-    sigmoid-gated product of :func:`gated_clamp_mul` in the epilogue.  ``relu2``: ``out = max(x @ w.T, 0)^2``."""
-    silu_mul = silu_mul or gated is not None
-    kind = 2 if gated is not None else (3 if relu2 else 0)
+    sigmoid-gated product of :func:`gated_clamp_mul` in the epilogue.  ``relu2``: ``out = max(x @ w.T, 0)^2``.  ``gelu_mul``: the
+    stacked weight with ``gelu_tanh(gate) * up``."""
+    silu_mul = silu_mul or gated is not None or gelu_mul
+    kind = 2 if gated is not None else (3 if relu2 else (4 if gelu_mul else 0))
     limit, slope, up_offset = gated if gated is not None else (0.0, 0.0, 0.0)
     need_cuda(x, w, bias, out)
     m, k = x.shape
@@ -359,7 +360,7 @@ def _num_sms(device) -> int:
 
 def gemm_tcgen05_tiles(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
                        silu_mul: bool = False, tile_width: int = 0, pairs: Optional[bool] = None,
-                       gated: Optional[tuple] = None, relu2: bool = False) -> None:
+                       gated: Optional[tuple] = None, relu2: bool = False, gelu_mul: bool = False) -> None:
     """``out = x @ w.T + bias`` for many rows: one persistent CTA per SM walks 128-row tiles, the accumulator
     double-buffered in TMEM so that the epilogue of a tile overlaps the products of the next.
 
@@ -368,11 +369,11 @@ def gemm_tcgen05_tiles(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Te
     the call when 0.  ``pairs``: two SMs share a 256-row tile and each loads only half of its weight rows
     (``cta_group::2``); the default for more than 128 rows.  ``gated = (limit, slope, up_offset)``: the stacked weight
     with the clamped, sigmoid-gated product of :func:`gated_clamp_mul` in the epilogue; ``relu2``: ``out = max(x @ w.T,
-    0)^2``.
+    0)^2``; ``gelu_mul``: the stacked weight with ``gelu_tanh(gate) * up``.
     """
     need_cuda(x, w, bias, out)
-    silu_mul = silu_mul or gated is not None
-    epilogue = 2 if gated is not None else (3 if relu2 else (1 if silu_mul else 0))
+    silu_mul = silu_mul or gated is not None or gelu_mul
+    epilogue = 2 if gated is not None else (3 if relu2 else (4 if gelu_mul else (1 if silu_mul else 0)))
     limit, slope, up_offset = gated if gated is not None else (0.0, 0.0, 0.0)
     m, k = x.shape
     n = out.shape[1]
@@ -477,6 +478,24 @@ def linear_gated_clamp_mul(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.
     gated_clamp_mul(gate_up, out, *gated)
 
 
+def linear_gelu_mul(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor) -> None:
+    """``out = gelu_tanh(x @ gate.T) * (x @ up.T)`` with ``w_gate_up = [gate; up]`` stacked.  Where :func:`linear_silu_mul` runs
+    its activation in the product's epilogue this one does too, by the same rules; otherwise product, then
+    :func:`gated_gelu_mul`."""
+    need_cuda(x, w_gate_up, out)
+    if _small_m_ok(x, w_gate_up, fused="silu"):
+        gemm_smallm(x, w_gate_up, None, out, gelu_mul=True)
+        return
+    min_rows = TC_FUSED_MIN_ROWS_LARGE if w_gate_up.shape[0] * w_gate_up.shape[1] >= TC_FUSED_LARGE_ELEMENTS else TC_FUSED_MIN_ROWS
+    if x.shape[0] >= min_rows and out.dtype == torch.bfloat16 and _tc_ok(x, w_gate_up, None, out):
+        gemm_tcgen05_tiles(x, w_gate_up, None, out, gelu_mul=True)
+        _tc_launched[x.device] = True
+        return
+    gate_up = torch.empty((x.shape[0], w_gate_up.shape[0]), dtype=out.dtype, device=x.device)
+    linear(x, w_gate_up, None, gate_up)
+    gated_gelu_mul(gate_up, out)
+
+
 def linear_relu2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     """``out = max(x @ w.T, 0)^2``: the activation in the product's epilogue on the weight-streaming kernel (up to 16
     rows) and on the tcgen05 kernel (from ``TC_FUSED_MIN_ROWS`` rows); otherwise product, then :func:`relu2`."""
@@ -567,13 +586,32 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: 
     gemm_nt(x, w, bias, out)
 
 
+def _mask_code(window: Optional[int], chunk: Optional[int]) -> int:
+    """How the kernels take a layer's mask: a window as itself, chunks as minus their size, neither as 0."""
+    if window and chunk:
+        raise KernelError("attention: a layer has a window or chunks, not both")
+    return int(window) if window else -int(chunk or 0)
+
+
+def _bias_args(bias: Optional[torch.Tensor], n_heads: int):
+    if bias is None:
+        return ptr(None), c_int(0)
+    if bias.dtype != torch.float32 or bias.dim() != 2 or bias.shape[0] != n_heads or not bias.is_contiguous() or not bias.is_cuda:
+        raise KernelError(f"attention: the bias by distance must be contiguous float32 [{n_heads}, distances] on the device")
+    return ptr(bias), c_int(bias.shape[1])
+
+
 def paged_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, tables: torch.Tensor,
                     tok_seg: torch.Tensor, pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                     page_size: int, page_stride: int, kv_stride: int, window: Optional[int], scale: float,
-                    sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
+                    sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
+                    chunk: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of each token over its request's cache pages (general kernel).  ``kv_stride`` 0: the cache has
     one plane whose rows are keys and values at once.  ``sinks``: float32, one per query head; ``exp(sinks[h])`` joins
-    the softmax's denominator (a term without key and value).  ``softcap`` c: a scaled score s becomes ``c tanh(s / c)``."""
+    the softmax's denominator (a term without key and value).  ``softcap`` c: a scaled score s becomes ``c tanh(s / c)``.
+    ``chunk``: a query sees the keys of its own chunk of that many positions, chunks counted from position 0 (``window`` is
+    then None).  ``bias``: float32 ``[n_heads, distances]``; entry ``[h, min(i - j, distances - 1)]`` joins the score of query i
+    and key j, after the scale and the cap."""
     need_cuda(q, cache, out, tables, tok_seg, pos, sinks)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != n_heads or not sinks.is_contiguous()):
         raise KernelError(f"paged_attention: sinks must be contiguous float32 with {n_heads} entries")
@@ -585,7 +623,7 @@ def paged_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, tab
     _attention_generic.call("zi_paged_attention", ptr(q), ptr(cache), ptr(out), c_int(dtype_code(q.dtype)),
                             ptr(tables), ptr(tok_seg), ptr(pos), c_int(n), c_int(n_heads), c_int(n_kv_heads),
                             c_int(head_dim), c_int(page_size), c_int(tables.shape[1]), c_ll(page_stride),
-                            c_ll(kv_stride), c_int(window or 0), c_float(scale), ptr(sinks), c_float(softcap or 0.0), stream())
+                            c_ll(kv_stride), c_int(_mask_code(window, chunk)), c_float(scale), ptr(sinks), c_float(softcap or 0.0), *_bias_args(bias, n_heads), stream())
 
 
 PREFILL_TILE_ROWS = 128          # query rows per entry of a step's tile list
@@ -599,7 +637,8 @@ def _check_sinks(sinks: Optional[torch.Tensor], n_heads: int) -> None:
 def decode_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, tables: torch.Tensor,
                      tok_seg: torch.Tensor, pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                      page_size: int, page_stride: int, kv_stride: int, window: Optional[int], scale: float,
-                     sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
+                     sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
+                     chunk: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     """One query token per request, bfloat16, tensor cores; a cluster of eight thread blocks per
     (request, key/value head) shares the context and merges through distributed shared memory.  ``kv_stride`` 0 and
     ``sinks`` and ``softcap``: as :func:`paged_attention`."""
@@ -612,8 +651,8 @@ def decode_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, ta
         raise KernelError("decode_attention: bfloat16 only")
     _attention_mma.call("zi_decode_attention", ptr(q), ptr(cache), ptr(out), ptr(tables), ptr(tok_seg), ptr(pos),
                         c_int(n), c_int(n_heads), c_int(n_kv_heads), c_int(head_dim), c_int(page_size),
-                        c_int(tables.shape[1]), c_ll(page_stride), c_ll(kv_stride), c_int(window or 0),
-                        c_float(scale), ptr(sinks), c_float(softcap or 0.0), stream())
+                        c_int(tables.shape[1]), c_ll(page_stride), c_ll(kv_stride), c_int(_mask_code(window, chunk)),
+                        c_float(scale), ptr(sinks), c_float(softcap or 0.0), *_bias_args(bias, n_heads), stream())
 
 
 def decode_attention_split_from() -> int:
@@ -625,7 +664,8 @@ def decode_attention_split_from() -> int:
 def decode_attention_tma(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, tables: torch.Tensor,
                          tok_seg: Optional[torch.Tensor], pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                          page_size: int, page_stride: int, kv_stride: int, window: Optional[int], scale: float,
-                         max_kv_len: int = 0, sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
+                         max_kv_len: int = 0, sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
+                         chunk: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     """One query token per request, bfloat16: the cluster kernel with 32-key tiles dealt to single warps, each
     fed by TMA through the block table into a ring of its own.  Same arguments as :func:`decode_attention`;
     head_dim 64 or 128, pages of a power of two from 8 to 128 tokens.  ``max_kv_len``: an upper bound of the cached
@@ -652,15 +692,16 @@ def decode_attention_tma(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
     _attention_mma.call("zi_decode_attention_tma", ptr(q), ptr(cache), ptr(out), ptr(tables), ptr(tok_seg), ptr(pos),
                         ptr(_tc_status(q.device)), c_int(q.shape[0]), c_int(n_heads), c_int(n_kv_heads), c_int(head_dim),
                         c_int(page_size), c_int(tables.shape[1]), c_ll(cache.shape[0]), c_ll(page_stride), c_ll(kv_stride),
-                        c_int(window or 0), c_float(scale), c_int(int(max_kv_len) if part_floats else 0), ptr(part),
-                        c_ll(part_floats), ptr(sinks), c_float(softcap or 0.0), stream())
+                        c_int(_mask_code(window, chunk)), c_float(scale), c_int(int(max_kv_len) if part_floats else 0), ptr(part),
+                        c_ll(part_floats), ptr(sinks), c_float(softcap or 0.0), *_bias_args(bias, n_heads), stream())
     _tc_launched[q.device] = True
 
 
 def prefill_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, tables: torch.Tensor,
                       tiles: torch.Tensor, pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                       page_size: int, page_stride: int, kv_stride: int, window: Optional[int], scale: float,
-                      sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
+                      sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
+                      chunk: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     """Portions of prompts, bfloat16, ``mma.sync`` tensor-core path.  ``tiles`` int32 ``[n_tiles, 3]``: (first token,
     rows <= 128, segment); the positions of a tile's tokens are consecutive.  Takes any page size and windows."""
     need_cuda(q, cache, out, tables, tiles, pos)
@@ -670,14 +711,15 @@ def prefill_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, t
         raise KernelError("prefill_attention: bfloat16 only")
     _attention_mma.call("zi_prefill_attention", ptr(q), ptr(cache), ptr(out), ptr(tables), ptr(tiles), ptr(pos),
                         c_int(tiles.shape[0]), c_int(n_heads), c_int(n_kv_heads), c_int(head_dim), c_int(page_size),
-                        c_int(tables.shape[1]), c_ll(page_stride), c_ll(kv_stride), c_int(window or 0),
-                        c_float(scale), ptr(sinks), c_float(softcap or 0.0), stream())
+                        c_int(tables.shape[1]), c_ll(page_stride), c_ll(kv_stride), c_int(_mask_code(window, chunk)),
+                        c_float(scale), ptr(sinks), c_float(softcap or 0.0), *_bias_args(bias, n_heads), stream())
 
 
 def prefill_attention_tcgen05(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, tables: torch.Tensor,
                               tiles: torch.Tensor, pos: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                               page_size: int, page_stride: int, kv_stride: int, window: Optional[int], scale: float,
-                              sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None) -> None:
+                              sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
+                              chunk: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     """Portions of prompts, bfloat16, on tcgen05: scores and outputs accumulate in TMEM, K and V pages arrive by
     TMA through the block table.  Same arguments as :func:`prefill_attention`; head_dim 64 or 128, pages of a power
     of two from 8 to 128 tokens.  A bounded wait that runs out is reported by :func:`tcgen05_status`."""
@@ -689,8 +731,8 @@ def prefill_attention_tcgen05(q: torch.Tensor, cache: torch.Tensor, out: torch.T
     _attention_tcgen05.call("zi_prefill_attention_tcgen05", ptr(q), ptr(cache), ptr(out), ptr(tables), ptr(tiles), ptr(pos),
                             ptr(_tc_status(q.device)), c_int(q.shape[0]), c_int(tiles.shape[0]), c_int(n_heads),
                             c_int(n_kv_heads), c_int(head_dim), c_int(page_size), c_int(tables.shape[1]),
-                            c_ll(cache.shape[0]), c_ll(page_stride), c_ll(kv_stride), c_int(window or 0), c_float(scale), ptr(sinks),
-                            c_float(softcap or 0.0), stream())
+                            c_ll(cache.shape[0]), c_ll(page_stride), c_ll(kv_stride), c_int(_mask_code(window, chunk)), c_float(scale), ptr(sinks),
+                            c_float(softcap or 0.0), *_bias_args(bias, n_heads), stream())
     _tc_launched[q.device] = True
 
 
@@ -703,7 +745,7 @@ LATENT_TENSOR_CORES = True       # one-plane caches and sinks on the tensor-core
 
 def attention(q: torch.Tensor, cache, out: torch.Tensor, ctx, n_heads: int, n_kv_heads: int, head_dim: int,
               window: Optional[int], scale: float, sinks: Optional[torch.Tensor] = None,
-              softcap: Optional[float] = None) -> None:
+              softcap: Optional[float] = None, chunk: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
     """Attention of a step's tokens over the cache (``cache`` is a CallCacheView, ``ctx`` a StepContext).
 
     Picks a kernel by dtype and by the shape of the step; all of them compute the same function.
@@ -711,7 +753,8 @@ def attention(q: torch.Tensor, cache, out: torch.Tensor, ctx, n_heads: int, n_kv
     of a mixed step, on the cluster decode kernel, anything else on the tcgen05 prefill kernel (pages of 8..128 tokens) or the ``mma.sync`` prefill kernel (other
     page sizes); float32 and other head sizes on the general kernel.  ``sinks`` (float32, one per query head) and a cache
     with one plane (``cache.kv_stride`` 0, rows that are keys and values at once) are taken by every kernel, and so is
-    ``softcap`` (scores through ``c tanh(s / c)``).
+    ``softcap`` (scores through ``c tanh(s / c)``), ``chunk`` (a mask by chunks of positions) and ``bias`` (a number per head and
+    distance that joins the score).
     """
     tables = ctx.tables[cache.group]
     if (q.dtype == torch.bfloat16 and head_dim in (64, 128)
@@ -721,11 +764,11 @@ def attention(q: torch.Tensor, cache, out: torch.Tensor, ctx, n_heads: int, n_kv
             # in a step of single tokens, token n is segment n
             decode_attention_tma(q, cache.tensor, out, tables, None, ctx.positions, n_heads, n_kv_heads, head_dim,
                                  cache.page_size, cache.page_stride, cache.kv_stride, window, scale,
-                                 max_kv_len=min(ctx.max_kv_len, window) if window else ctx.max_kv_len, sinks=sinks, softcap=softcap)
+                                 max_kv_len=min(ctx.max_kv_len, window or chunk) if window or chunk else ctx.max_kv_len, sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
             return
         if ctx.decode_only:
             decode_attention(q, cache.tensor, out, tables, ctx.tok_seg, ctx.positions, n_heads, n_kv_heads, head_dim,
-                             cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap)
+                             cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
             return
         tiles = ctx.extras.get("attn_tiles")
         lead = ctx.extras.get("leading_singles", 0) if tiles is not None else 0
@@ -733,21 +776,21 @@ def attention(q: torch.Tensor, cache, out: torch.Tensor, ctx, n_heads: int, n_kv
             if tcgen05_attention_ok(head_dim, cache.page_size):     # the leading single tokens are segments 0 .. lead - 1
                 decode_attention_tma(q[:lead], cache.tensor, out[:lead], tables, None, ctx.positions[:lead], n_heads,
                                      n_kv_heads, head_dim, cache.page_size, cache.page_stride, cache.kv_stride, window, scale,
-                                     sinks=sinks, softcap=softcap)
+                                     sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
             else:
                 decode_attention(q[:lead], cache.tensor, out[:lead], tables, ctx.tok_seg[:lead], ctx.positions[:lead], n_heads,
                                  n_kv_heads, head_dim, cache.page_size, cache.page_stride, cache.kv_stride, window, scale,
-                                 sinks=sinks, softcap=softcap)
+                                 sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
         if tiles is not None and tcgen05_attention_ok(head_dim, cache.page_size):
             prefill_attention_tcgen05(q, cache.tensor, out, tables, tiles, ctx.positions, n_heads, n_kv_heads, head_dim,
-                                      cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap)
+                                      cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
             return
         if tiles is not None:
             prefill_attention(q, cache.tensor, out, tables, tiles, ctx.positions, n_heads, n_kv_heads, head_dim,
-                              cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap)
+                              cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
             return
     paged_attention(q, cache.tensor, out, tables, ctx.tok_seg, ctx.positions, n_heads, n_kv_heads,
-                    head_dim, cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap)
+                    head_dim, cache.page_size, cache.page_stride, cache.kv_stride, window, scale, sinks=sinks, softcap=softcap, chunk=chunk, bias=bias)
 
 
 def argmax(logits: torch.Tensor, out: torch.Tensor) -> None:
@@ -883,6 +926,16 @@ def gated_clamp_mul(gate_up: torch.Tensor, out: torch.Tensor, limit: float, slop
         raise KernelError(f"gated_clamp_mul: gate_up {tuple(gate_up.shape)} vs out {tuple(out.shape)}")
     _rowwise.call("zi_gated_clamp_mul", ptr(gate_up), ptr(out), c_int(dtype_code(out.dtype)), c_int(rows), c_int(two_i // 2),
                   c_float(limit), c_float(slope), c_float(up_offset), stream())
+
+
+def gated_gelu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
+    """``gate_up`` is ``[rows, 2 * I]`` (gate columns, then up columns): ``out = gelu_tanh(gate) * up``."""
+    need_cuda(gate_up, out)
+    need_contiguous("gate_up", gate_up), need_contiguous("out", out)
+    rows, two_i = gate_up.shape
+    if two_i % 2 or out.shape != (rows, two_i // 2) or out.dtype != gate_up.dtype:
+        raise KernelError(f"gated_gelu_mul: gate_up {tuple(gate_up.shape)} vs out {tuple(out.shape)}")
+    _rowwise.call("zi_gated_gelu_mul", ptr(gate_up), ptr(out), c_int(dtype_code(out.dtype)), c_int(rows), c_int(two_i // 2), stream())
 
 
 def rmsnorm_append(x: torch.Tensor, w: torch.Tensor, eps: float, cache: torch.Tensor, tables: torch.Tensor,
@@ -1320,6 +1373,94 @@ def rotary_norm(x: torch.Tensor, q_out: torch.Tensor, pos: torch.Tensor, inv_fre
                   c_ll(cache.kv_stride if cache is not None else 0), stream())
 
 
+QK_NORMS = {None: 0, "head": 1, "row": 2}
+
+
+def qk_norm_append(x: torch.Tensor, q_out: torch.Tensor, pos: torch.Tensor, cache, tables: torch.Tensor, tok_seg: Optional[torch.Tensor],
+                   n_q: int, n_k: int, qk_dim: int, v_dim: int, row_dim: int, norm: Optional[str] = None, qw: Optional[torch.Tensor] = None,
+                   kw: Optional[torch.Tensor] = None, eps: float = 0.0, inv_freq: Optional[torch.Tensor] = None, mag: float = 1.0,
+                   rot_dims: int = 0, interleaved: bool = False, heat: Optional[tuple] = None, v_first: Optional[torch.Tensor] = None,
+                   lam: float = 0.0) -> None:
+    """Queries, keys and values of a step's tokens made ready for attention.  ``x`` ``[tokens, (n_q + n_k) * qk_dim + n_k * v_dim
+    (+ more)]`` (rows may be strided).  ``norm``: ``"head"``: every query and key head is divided by its root mean square and
+    multiplied by a weight that the heads share (float32 ``[qk_dim]``); ``"row"``: the same over a token's whole query row and
+    whole key row (weights of that many entries); None: not.  Then the first ``rot_dims`` entries of every query and key head
+    turn by position (as :func:`rotary`; cosines and sines times ``mag``), then queries are multiplied by ``1 + c ln(floor((pos +
+    1) / every) + 1)`` (``heat = (c, every)``).  ``v_first`` (``[tokens, n_k * v_dim]``, rows may be strided): values become
+    ``(1 - lam) v + lam v_first``.  Queries go to ``q_out`` ``[tokens, n_q, row_dim]``, keys and values to the two planes of
+    ``cache`` (a CallCacheView); what lies past a head's own entries is written as zero."""
+    need_cuda(x, q_out, pos, tables, tok_seg, qw, kw, inv_freq, v_first)
+    need_int32("pos", pos), need_int32("tables", tables)
+    need_contiguous("q_out", q_out)
+    n = x.shape[0]
+    ct = cache.tensor
+    if (x.stride(1) != 1 or q_out.dtype != x.dtype or q_out.numel() != n * n_q * row_dim or x.shape[1] < (n_q + n_k) * qk_dim + n_k * v_dim
+            or ct.dtype != x.dtype or ct.shape[-1] != row_dim):
+        raise KernelError("qk_norm_append: x, q_out and the cache do not agree")
+    if norm not in QK_NORMS:
+        raise KernelError(f"qk_norm_append: norm={norm!r} is not 'head', 'row' or None")
+    if norm is not None:
+        for name, t, count in (("qw", qw, n_q * qk_dim if norm == "row" else qk_dim), ("kw", kw, n_k * qk_dim if norm == "row" else qk_dim)):
+            if t is None or t.dtype != torch.float32 or t.numel() != count or not t.is_contiguous():
+                raise KernelError(f"qk_norm_append: {name} must be contiguous float32 with {count} entries")
+    if rot_dims and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2 or not inv_freq.is_contiguous()):
+        raise KernelError(f"qk_norm_append: inv_freq must be float32 with {rot_dims // 2} entries")
+    if v_first is not None and (v_first.dtype != x.dtype or v_first.shape != (n, n_k * v_dim) or v_first.stride(1) != 1):
+        raise KernelError(f"qk_norm_append: v_first must be [{n}, {n_k * v_dim}] of x's type")
+    coef, every = heat if heat is not None else (0.0, 0.0)
+    _rowwise.call("zi_qk_norm_append", ptr(x), c_int(dtype_code(x.dtype)), c_ll(x.stride(0)), ptr(q_out), ptr(ct), ptr(tables), ptr(tok_seg),
+                  ptr(pos), ptr(qw), ptr(kw), c_int(QK_NORMS[norm]), c_float(eps), ptr(inv_freq), c_float(mag), c_int(rot_dims),
+                  c_int(1 if interleaved else 0), c_float(coef), c_float(every), ptr(v_first),
+                  c_ll(v_first.stride(0) if v_first is not None else 0), c_float(lam), c_int(n), c_int(n_q), c_int(n_k), c_int(qk_dim),
+                  c_int(v_dim), c_int(row_dim), c_int(cache.page_size), c_int(tables.shape[1]), c_ll(cache.page_stride),
+                  c_ll(cache.kv_stride), stream())
+
+
+def branches_rmsnorm(h: torch.Tensor, y: Optional[torch.Tensor], f: Optional[torch.Tensor], w: torch.Tensor, eps: float, out: torch.Tensor,
+                     row_idx: Optional[torch.Tensor] = None, write_h: bool = True, join=None) -> None:
+    """Branches that read the same input join the float32 stream ``h`` together, and the next norm follows: ``v = h + (y + f)``,
+    ``h = v`` where ``write_h``, ``out = v / sqrt(mean(v^2) + eps) * w`` (``w`` float32).  ``y`` and ``f`` may each be None, or float32
+    partial sums ``[parts, rows, hidden]`` (:func:`linear_for_residual`).  ``join = (y2, w1, w2, join_eps)``: the first branch is
+    two outputs joined on the way, ``(U(y) * w1 + U(y2) * w2) / 2``, ``U(u) = u / sqrt(mean(u^2) + join_eps)`` over a row, float32
+    weights.  With ``row_idx`` output row r comes from row ``row_idx[r]`` and ``h`` is left as it is."""
+    need_cuda(h, y, f, w, out, row_idx)
+    need_contiguous("h", h), need_contiguous("out", out)
+    if h.dtype != torch.float32 or h.dim() != 2:
+        raise KernelError(f"branches_rmsnorm: the stream must be float32 [rows, hidden], got {tuple(h.shape)} {h.dtype}")
+    hidden = h.shape[1]
+    if row_idx is not None:
+        need_int32("row_idx", row_idx), need_contiguous("row_idx", row_idx)
+        write_h = False
+    rows = row_idx.numel() if row_idx is not None else h.shape[0]
+    if out.shape != (rows, hidden):
+        raise KernelError(f"branches_rmsnorm: out {tuple(out.shape)} does not fit {(rows, hidden)}")
+
+    def parts_of(name, t):
+        if t is None:
+            return 0
+        need_contiguous(name, t)
+        if t.dim() == 3:
+            if t.dtype != torch.float32 or t.shape[1:] != h.shape:
+                raise KernelError(f"branches_rmsnorm: partial sums {name} {tuple(t.shape)} {t.dtype} vs {tuple(h.shape)}")
+            return t.shape[0]
+        if t.shape != h.shape or t.dtype != out.dtype:
+            raise KernelError(f"branches_rmsnorm: {name} {tuple(t.shape)} {t.dtype} vs {tuple(h.shape)} {out.dtype}")
+        return 0
+
+    y_parts, f_parts = parts_of("y", y), parts_of("f", f)
+    y2, w1, w2, join_eps = join if join is not None else (None, None, None, 0.0)
+    if join is not None:
+        need_cuda(y2, w1, w2)
+        if y is None or y_parts or parts_of("y2", y2):
+            raise KernelError("branches_rmsnorm: two joined outputs are both whole rows")
+    for name, t in (("w", w), ("w1", w1), ("w2", w2)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != hidden or not t.is_contiguous()):
+            raise KernelError(f"branches_rmsnorm: {name} must be contiguous float32 with {hidden} entries")
+    _rowwise.call("zi_branches_rmsnorm", ptr(h), ptr(y), c_int(y_parts), ptr(y2), ptr(f), c_int(f_parts), c_ll(h.shape[0] * hidden),
+                  c_int(dtype_code(out.dtype)), ptr(w1), ptr(w2), c_float(join_eps), ptr(w), c_float(eps), ptr(out), ptr(row_idx),
+                  c_int(rows), c_int(hidden), c_int(1 if write_h else 0), stream())
+
+
 def norm_add(h: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, rounded: Optional[torch.Tensor] = None) -> None:
     """``h += y / sqrt(mean(y^2) + eps) * w`` row by row, in float32 (``h`` float32 ``[rows, hidden]``); ``rounded`` (of y's
     type) receives the new ``h``."""
@@ -1346,7 +1487,7 @@ def gelu_mul_rows(t: torch.Tensor, table: torch.Tensor, col0: int, ids: torch.Te
 
 
 # ---- linear recurrences with a matrix state per head, csrc/linrec.cu ---------------------------------------------------------
-LINEAR_STATE_RULES = {"delta": 0, "decay": 1, "forget": 2}
+LINEAR_STATE_RULES = {"delta": 0, "decay": 1, "forget": 2, "expgate": 3}
 _SILU_ON = {"q": 1, "k": 2, "v": 4}
 
 
@@ -1355,7 +1496,7 @@ def linear_state(rule: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, s
                  a: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None,
                  a_log: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None, act_silu=False,
                  q_scale: float = 1.0, unit_eps: float = 1e-6, work: Optional[torch.Tensor] = None,
-                 decay_per_head: bool = False) -> None:
+                 decay_per_head: bool = False, den: Optional[torch.Tensor] = None, gate_cap: float = 0.0) -> None:
     """Walk each segment's tokens in order through a float32 state ``S`` (``dim x vdim``) per head.
 
     ``rule="delta"``: ``S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` with ``q`` and ``k`` made unit vectors
@@ -1365,7 +1506,12 @@ def linear_state(rule: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, s
     ``rule="decay"``: ``S <- decay_h S + k v^T; o = S^T q`` (``decay`` float32 ``[heads]``; ``q`` times ``q_scale``).
     ``rule="forget"``: ``S <- diag(f) S + (1 - f) v^T; o = S^T q`` with ``f = l + (1 - l) sigmoid(a)`` per head and key entry
     (``a [tokens, heads * dim]``, the lower bounds ``l`` in ``dt_bias`` float32 ``[heads * dim]``; ``k`` is None, ``kv_heads``
-    equals ``heads``; ``q`` times ``q_scale``).  ``act_silu``: True: q, k and v pass through SiLU first; a string names which
+    equals ``heads``; ``q`` times ``q_scale``).  ``rule="expgate"``: ``m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T;
+    n <- e^(f + m - m') n + e^(i - m') k; o = S^T q`` with ``i = c tanh((a + dt_bias) / c)``, ``f = ln sigmoid(c tanh((b + a_log) /
+    c))`` per head (``a``, ``b`` ``[tokens, heads]``, the two biases float32 ``[heads]``, c = ``gate_cap``, ``q`` times ``q_scale``);
+    ``den`` (float32 ``[tokens, heads]``) receives ``max(|n . q|, e^-m') + 1e-6``, by which the read-out is to be divided.  A
+    request's state is then ``[heads, vdim + 1, dim]`` (the last column is n) and, behind it, m ``[heads, vdim + 1]`` (one copy
+    per column): :func:`linear_state_floats` says how many entries.  ``act_silu``: True: q, k and v pass through SiLU first; a string names which
     of them do (``"q"``, ``"qk"``, ...).  ``q``, ``k`` ``[tokens, kv_heads * dim]`` (head h reads
     query/key head ``h // (heads / kv_heads)``) and ``v [tokens, heads * vdim]`` may have strided rows; ``y`` float32
     ``[tokens, heads * vdim]``.  A request's state (``[heads, vdim, dim]``, the first entries of its slot of ``state``) is read
@@ -1375,7 +1521,7 @@ def linear_state(rule: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, s
     ``work`` (float32, at least :func:`linear_state_work_floats` entries): a first kernel makes every token's inputs ready
     there (all tokens and heads at once) and the walk only copies and walks, which pays for segments of many tokens; without
     it the walk makes its inputs ready itself.  A token's result has the same bits either way."""
-    need_cuda(q, k, v, state, slots, bounds, y, a, b, dt_bias, a_log, decay, work)
+    need_cuda(q, k, v, state, slots, bounds, y, a, b, dt_bias, a_log, decay, work, den)
     forget = rule == "forget"
     if forget:
         if k is not None or kv_heads != heads:
@@ -1391,21 +1537,28 @@ def linear_state(rule: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, s
             or v.shape != (n, heads * vdim) or not (q.dtype == k.dtype == v.dtype) or y.dtype != torch.float32
             or y.shape != (n, heads * vdim)):
         raise KernelError(f"linear_state: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)}, y {tuple(y.shape)} do not agree")
-    per_head = bool(decay_per_head) and rule == "delta"
+    per_head = (bool(decay_per_head) and rule == "delta") or rule == "expgate"
+    if den is not None and (den.dtype != torch.float32 or den.shape != (n, heads) or not den.is_contiguous()):
+        raise KernelError(f"linear_state: den must be contiguous float32 {(n, heads)}")
     for name, t, width in (("a", a, heads if per_head else heads * dim), ("b", b, heads)):
         if t is not None and (t.shape != (n, width) or t.stride(1) != 1 or t.dtype != q.dtype):
             raise KernelError(f"linear_state: {name} must be [tokens, {width}] of q's type")
     for name, t, count in (("dt_bias", dt_bias, heads if per_head else heads * dim), ("a_log", a_log, heads), ("decay", decay, heads)):
         if t is not None and (t.dtype != torch.float32 or t.numel() != count or not t.is_contiguous()):
             raise KernelError(f"linear_state: {name} must be contiguous float32 with {count} entries")
-    if state.shape[1] < heads * vdim * dim:
+    if state.shape[1] < linear_state_floats(rule, heads, dim, vdim):
         raise KernelError("linear_state: the state slots are too small")
     sp, ss = _state_args(state, 0)
     _linrec.call("zi_linear_state", c_int(LINEAR_STATE_RULES[rule]), ptr(q), c_ll(q.stride(0)), ptr(k), c_ll(k.stride(0)), ptr(v),
                  c_ll(v.stride(0)), ptr(a), c_ll(a.stride(0) if a is not None else 0), ptr(b), c_ll(b.stride(0) if b is not None else 0),
                  c_int(dtype_code(q.dtype)), ptr(dt_bias), ptr(a_log), ptr(decay), sp, ss, ptr(slots), ptr(bounds), ptr(y), c_int(n),
                  c_int(n_segments), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(silu_bits), c_int(1 if per_head else 0),
-                 c_float(q_scale), c_float(unit_eps), ptr(work), c_ll(work.numel() if work is not None else 0), stream())
+                 c_float(q_scale), c_float(unit_eps), ptr(den), c_float(gate_cap), ptr(work), c_ll(work.numel() if work is not None else 0), stream())
+
+
+def linear_state_floats(rule: str, heads: int, dim: int, vdim: int) -> int:
+    """Entries of a request's float32 state for :func:`linear_state`."""
+    return heads * (vdim + 1) * (dim + 1) if rule == "expgate" else heads * vdim * dim
 
 
 def linear_state_work_floats(rule: str, n_tokens: int, heads: int, dim: int, vdim: int) -> int:
@@ -1413,26 +1566,30 @@ def linear_state_work_floats(rule: str, n_tokens: int, heads: int, dim: int, vdi
     and head a record of q, k (and the decays in the delta rule) padded to the kernel's 32, 64, 128 or 256 entries plus
     four scalars, and the values padded to whole tiles of 16 columns."""
     padded = 32 if dim <= 32 else 64 if dim <= 64 else 128 if dim <= 128 else 256
-    record = (2 if rule == "decay" else 3) * padded + 4
-    return n_tokens * heads * (record + (vdim + 15) // 16 * 16)
+    record = (2 if rule in ("decay", "expgate") else 3) * padded + 4
+    columns = vdim + 1 if rule == "expgate" else vdim
+    return n_tokens * heads * (record + (columns + 15) // 16 * 16)
 
 
 GROUP_NORM_GATES = {"sigmoid": 0, "silu": 1, None: 2}
 
 
 def group_rmsnorm_gate(y: torch.Tensor, z: Optional[torch.Tensor], w: torch.Tensor, n_groups: int, eps: float, out: torch.Tensor,
-                       gate: Optional[str] = "sigmoid") -> None:
+                       gate: Optional[str] = "sigmoid", den: Optional[torch.Tensor] = None) -> None:
     """``out = unit_rms(y) * w * gate(z)`` with the root mean square over each of ``n_groups`` equal parts of a row and
     ``w`` repeated along the row when it is shorter; ``y`` float32, ``z`` (rows may be strided) and ``out`` of the step's type.
-    ``gate``: ``"sigmoid"``, ``"silu"`` or None (no gate; ``z`` is then None)."""
-    need_cuda(y, z, w, out)
+    ``gate``: ``"sigmoid"``, ``"silu"`` or None (no gate; ``z`` is then None).  ``den`` (float32 ``[rows, n_groups]``): every group
+    of ``y`` is divided by its own number first."""
+    need_cuda(y, z, w, out, den)
+    if den is not None and (den.dtype != torch.float32 or den.shape != (y.shape[0], n_groups) or not den.is_contiguous()):
+        raise KernelError(f"group_rmsnorm_gate: den must be contiguous float32 {(y.shape[0], n_groups)}")
     need_contiguous("y", y), need_contiguous("w", w), need_contiguous("out", out)
     n, inner = y.shape
     if gate not in GROUP_NORM_GATES or (gate is None) != (z is None):
         raise KernelError(f"group_rmsnorm_gate: gate={gate!r} is not 'sigmoid', 'silu' or None, or does not fit z")
     if y.dtype != torch.float32 or out.shape != (n, inner) or (z is not None and (z.shape != (n, inner) or z.stride(1) != 1 or out.dtype != z.dtype)):
         raise KernelError(f"group_rmsnorm_gate: y {tuple(y.shape)}, z {tuple(z.shape) if z is not None else None}, out {tuple(out.shape)} do not agree")
-    _linrec.call("zi_group_rmsnorm_gate", ptr(y), ptr(z), c_int(dtype_code(out.dtype)), c_ll(z.stride(0) if z is not None else 0), ptr(w),
+    _linrec.call("zi_group_rmsnorm_gate", ptr(y), ptr(den), ptr(z), c_int(dtype_code(out.dtype)), c_ll(z.stride(0) if z is not None else 0), ptr(w),
                  c_int(dtype_code(w.dtype)), c_int(w.numel()), ptr(out), c_int(n), c_int(inner), c_int(n_groups), c_float(eps),
                  c_int(GROUP_NORM_GATES[gate]), stream())
 

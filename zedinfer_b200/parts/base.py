@@ -80,6 +80,9 @@ class ResidualStream:
     # float32 weight, the second one's, eps) for ``(U(delta) * w1 + U(second) * w2) / 2``, ``U`` the division by the root mean
     # square over a row; the joined row then passes ``delta_norm``.  None: ``delta`` is the whole branch
     delta_join: Optional[tuple] = None
+    # a second branch output that joins ``h`` together with ``delta`` (arrangements whose sublayers read the same normed input);
+    # like ``delta`` it may come as partial sums.  None: ``delta`` is all that is pending
+    delta_more: Optional[torch.Tensor] = None
     # ``h`` rounded to the step's type, where the kernel that last changed ``h`` made that copy on its way (arrangements
     # whose sublayers read the stream itself); whoever changes ``h`` otherwise sets it to None
     rounded: Optional[torch.Tensor] = None
@@ -87,7 +90,7 @@ class ResidualStream:
     def as_input(self, ctx: "StepContext") -> torch.Tensor:
         """The stream as a sublayer's input: ``h`` itself in a float32 step, else its rounded copy (made here if nobody
         has made it yet).  Nothing may be pending in ``delta``."""
-        if self.delta is not None:
+        if self.delta is not None or self.delta_more is not None:
             raise RuntimeError("a branch output is still pending: fold it into the stream first")
         if ctx.dtype == torch.float32:
             return self.h

@@ -9,7 +9,7 @@ stream until the next norm folds it into the float32 residual.
 sum in float32.  A layer without a feed-forward (no ``ffn``, no ``norm2``) is its first half alone.
 
 ``branch_norm`` puts the norm on each branch's output; ``sandwich_norm`` has one before and one after every sublayer and
-may run two mixers side by side on the same input."""
+may run two mixers side by side on the same input; ``shared_norm`` has one norm whose output every sublayer reads."""
 from __future__ import annotations
 
 from typing import Mapping
@@ -124,3 +124,44 @@ class SandwichNormBlock(Block):
         normed2 = ctx.empty(n, hidden)
         self.norms["norm2"].forward_residual(stream, normed2)
         stream.delta, stream.delta_norm, stream.delta_scale, stream.delta_join = self.ffn.forward(normed2, ctx), self.norms["norm2b"], 1.0, None
+
+
+@register_block("shared_norm")
+class SharedNormBlock(Block):
+    """One norm, and all sublayers read its output:
+
+        a = norm1(h);  h = h + (mixer(a) + ffn(a))
+
+    ``ffn`` is optional.  With a second mixer (role ``mixer2``, a cache of its own) the mixers' outputs are joined as in
+    ``sandwich_norm``: ``(U(y1) * w1 + U(y2) * w2) / 2`` with the weights of the norms ``mix_out`` and ``mix2_out`` (built with
+    ``float32_weight``) and their epsilon.  Both branches stay pending in the stream (``ResidualStream.delta``, ``delta_join``,
+    ``delta_more``) until the next layer's norm or the model's last one folds them: one kernel per layer besides the
+    sublayers' own (``ops.branches_rmsnorm``)."""
+    capture_safe = True
+
+    def __init__(self, parts):
+        super().__init__(parts)
+        have = self.parts()
+        need = ["mixer", "norm1"]
+        if any(role in have for role in ("mixer2", "mix_out", "mix2_out")):
+            need += ["mixer2", "mix_out", "mix2_out"]
+        missing = [role for role in need if role not in have]
+        if missing:
+            raise ValueError(f"the shared_norm arrangement needs the parts {missing} as well")
+        self.mixer2 = have.get("mixer2")
+        if self.mixer2 is not None and self.norms["mix_out"].eps != self.norms["mix2_out"].eps:
+            raise ValueError("the shared_norm arrangement joins two mixers with one epsilon")
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, caches: Mapping[str, CallCacheView],
+                owns_cache: bool) -> None:
+        n, hidden = stream.h.shape
+        normed = ctx.empty(n, hidden)
+        self.norms["norm1"].forward_residual(stream, normed)
+        stream.delta_scale, stream.delta_norm, stream.delta_join = 1.0, None, None
+        if self.mixer2 is None:
+            stream.delta = self.mixer.forward_for_residual(normed, ctx, caches["mixer"], owns_cache)
+        else:
+            stream.delta = self.mixer.forward(normed, ctx, caches["mixer"], owns_cache)
+            stream.delta_join = (self.mixer2.forward(normed, ctx, caches["mixer2"], owns_cache), self.norms["mix_out"].weight,
+                                 self.norms["mix2_out"].weight, self.norms["mix_out"].eps)
+        stream.delta_more = self.ffn.forward_for_residual(normed, ctx) if self.ffn is not None else None

@@ -18,13 +18,21 @@ the gate's inputs projected in one step each, and a SiLU gate: ``out = Wo (unit_
     per head:   S <- diag(f) S + (1 - f) v^T;   o = S^T q
     out = Wo (unit_rms_per_head(o) * w_norm)                                   w_norm [vdim], shared by heads
 
+``exp_gate`` (exponential input and forget gates per head, kept in range by a running maximum, and a key sum that the read-out
+is divided by: the matrix memory of xLSTM), with c the gates' cap:
+
+    q = Wq h / sqrt(dim);   k = Wk h;   v = Wv h;   i = c tanh((Wi h + bi) / c);   f = ln sigmoid(c tanh((Wf h + bf) / c))
+    per head:   m' = max(f + m, i);   S <- e^(f + m - m') S + e^(i - m') k v^T;   n <- e^(f + m - m') n + e^(i - m') k
+                o = S^T q / (max(|n . q|, e^-m') + 1e-6)                       S, n and m zero before the first token
+    out = Wo (unit_rms_per_head(o) * w_norm * sigmoid(Wg h))                                      w_norm [H * vdim]
+
 ``lightning`` (a constant decay per head):
 
     q, k, v = silu(Wq h), silu(Wk h), silu(Wv h);    per head   S <- decay_a S + k v^T;   o = S^T q
     out = Wo (unit_rms(concat(o)) * w_norm * sigmoid(Wg h))                                       w_norm [H * vdim]
 
 What a request carries from step to step is one slot of fixed-size float32 state: S of every head laid out ``[H, vdim,
-dim]`` and, for ``channel_delta``, the convolution's last ``taps - 1`` inputs behind it.  A step runs the tokens it brings
+dim]`` (``exp_gate``: with n and m, see ``ops.linear_state``) and, for ``channel_delta``, the convolution's last ``taps - 1`` inputs behind it.  A step runs the tokens it brings
 from that state and leaves the state behind its last token, so a prompt may be cut anywhere and a decoded token is a portion
 of one.  Unit vectors, sigmoid, softplus, decays, the state and every sum of the recurrence are float32 whatever the step's
 type; the projections, the convolution and the activations on them have the step's type.
@@ -243,6 +251,62 @@ class ForgetGateMixer(Mixer):
                          work=_walk_workspace("forget", ctx, n, self.heads, self.dim, self.vdim))
         normed = ctx.empty(n, self.inner)
         ops.group_rmsnorm_gate(y, None, self.g, self.heads, self.eps, normed, gate=None)
+        out = ctx.empty(n, self.hidden_size)
+        ops.linear(normed, self.w_o, None, out)
+        return out
+
+
+@register_mixer("exp_gate")
+class ExpGateMixer(Mixer):
+    capture_safe = True
+
+    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, gate_cap: float, eps: float,
+                 names: Optional[Mapping[str, str]] = None):
+        if min(hidden_size, heads, dim, vdim) <= 0:
+            raise ValueError("exp_gate: every size must be positive")
+        if dim > 256:
+            raise ValueError(f"exp_gate: dim={dim} is not supported; the recurrence kernel takes at most 256")
+        if not gate_cap > 0.0:
+            raise ValueError(f"exp_gate: gate_cap={gate_cap} must be positive")
+        self.hidden_size, self.heads, self.dim, self.vdim, self.eps = int(hidden_size), int(heads), int(dim), int(vdim), float(eps)
+        self.gate_cap = float(gate_cap)
+        self.qk_width, self.inner = self.heads * self.dim, self.heads * self.vdim
+        self.names = {"q": "q", "k": "k", "v": "v", "g": "g", "i": "i", "i_bias": "i.b", "f": "f", "f_bias": "f.b", "norm": "norm", "o": "o"}
+        self.names.update(names or {})
+        self.w_in = self.i_bias = self.f_bias = self.g = self.w_o = None
+        self._offsets: List[int] = []
+
+    def cache_need(self):
+        return StateNeed((ops.linear_state_floats("expgate", self.heads, self.dim, self.vdim),), torch.float32)
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        nm, h = self.names, self.hidden_size
+        return {nm["q"]: TensorSpec((self.qk_width, h)), nm["k"]: TensorSpec((self.qk_width, h)), nm["v"]: TensorSpec((self.inner, h)),
+                nm["g"]: TensorSpec((self.inner, h)), nm["i"]: TensorSpec((self.heads, h)), nm["i_bias"]: TensorSpec((self.heads,)),
+                nm["f"]: TensorSpec((self.heads, h)), nm["f_bias"]: TensorSpec((self.heads,)),
+                nm["norm"]: TensorSpec((self.inner,), init=("one_plus_normal", 0.01)), nm["o"]: TensorSpec((h, self.inner))}
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        nm = self.names
+        self.w_in, self._offsets = _stack_padded([tensors[nm[r]] for r in ("q", "k", "v", "g", "i", "f")])
+        self.i_bias, self.f_bias = tensors[nm["i_bias"]].float().contiguous(), tensors[nm["f_bias"]].float().contiguous()   # float32: they enter the recurrence
+        self.g, self.w_o = tensors[nm["norm"]].contiguous(), tensors[nm["o"]].contiguous()
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CallCacheView, owns_cache: bool) -> torch.Tensor:
+        state = _state_and_slots(cache, ctx, owns_cache, "an exponential-gate mixer")
+        n = x.shape[0]
+        proj = ctx.empty(n, self.w_in.shape[0])
+        ops.linear(x, self.w_in, None, proj)
+        o_q, o_k, o_v, o_g, o_i, o_f = self._offsets
+        y = ctx.empty(n, self.inner, dtype=torch.float32)
+        den = ctx.empty(n, self.heads, dtype=torch.float32)
+        ops.linear_state("expgate", proj[:, o_q:o_q + self.qk_width], proj[:, o_k:o_k + self.qk_width], proj[:, o_v:o_v + self.inner], state,
+                         ctx.slots, step_segment_bounds(ctx), y, ctx.n_segments, self.heads, self.heads, self.dim, self.vdim,
+                         a=proj[:, o_i:o_i + self.heads], b=proj[:, o_f:o_f + self.heads], dt_bias=self.i_bias, a_log=self.f_bias,
+                         q_scale=self.dim ** -0.5, den=den, gate_cap=self.gate_cap,
+                         work=_walk_workspace("expgate", ctx, n, self.heads, self.dim, self.vdim))
+        normed = ctx.empty(n, self.inner)
+        ops.group_rmsnorm_gate(y, proj[:, o_g:o_g + self.inner], self.g, self.heads, self.eps, normed, den=den)
         out = ctx.empty(n, self.hidden_size)
         ops.linear(normed, self.w_o, None, out)
         return out

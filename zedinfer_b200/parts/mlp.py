@@ -1,4 +1,4 @@
-"""Gated feed-forward: ``down(up(x) * act(gate(x)))`` with SiLU, no biases unless asked
+"""Gated feed-forward: ``down(up(x) * act(gate(x)))`` with SiLU (or the tanh form of GELU), no biases unless asked
 (src/frontend/models/transformer_forward.cpp:128-137, src/backend/ops/swiglu/cpu/swiglu_cpu.cpp:13-20).
 Gate and up weights are stacked at load so one product makes both."""
 from __future__ import annotations
@@ -26,8 +26,9 @@ class GatedMLP(FeedForward):
                  names: Optional[Mapping[str, str]] = None):
         """``names``: the local tensor names of the three weights by role (``gate``, ``up``, ``down``); a bias is the
         weight's name with ``.weight`` replaced by ``.bias``."""
-        if activation != "silu":
-            raise ValueError(f"gated_mlp: activation {activation!r} is not supported (only 'silu')")
+        if activation not in ("silu", "gelu_tanh") or (bias and activation != "silu"):
+            raise ValueError(f"gated_mlp: activation {activation!r} is not supported (only 'silu', or 'gelu_tanh' without biases)")
+        self.activation = activation
         if hidden_size <= 0 or intermediate_size <= 0:
             raise ValueError("gated_mlp: sizes must be positive")
         self.hidden_size, self.intermediate_size, self.bias = int(hidden_size), int(intermediate_size), bool(bias)
@@ -61,7 +62,10 @@ class GatedMLP(FeedForward):
 
     def _activation(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         act = ctx.empty(x.shape[0], self.intermediate_size)
-        ops.linear_silu_mul(x, self.w_gate_up, self.b_gate_up, act)     # activation in the product's epilogue where it can be
+        if self.activation == "gelu_tanh":
+            ops.linear_gelu_mul(x, self.w_gate_up, act)
+        else:
+            ops.linear_silu_mul(x, self.w_gate_up, self.b_gate_up, act)     # activation in the product's epilogue where it can be
         return act
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:

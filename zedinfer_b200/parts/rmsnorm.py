@@ -40,8 +40,15 @@ class RMSNorm(Norm):
 
     def forward_residual(self, stream: ResidualStream, out: torch.Tensor,
                          row_idx: Optional[torch.Tensor] = None) -> None:
-        if stream.delta is not None and (stream.delta_norm is not None or stream.delta_join is not None):
+        if stream.delta is not None and stream.delta_norm is not None:
             raise RuntimeError("rmsnorm cannot fold a branch output that must pass a norm of its own first")
+        if stream.delta_more is not None or (stream.delta is not None and stream.delta_join is not None):
+            if not self.float32_weight or stream.delta_scale != 1.0:
+                raise RuntimeError("rmsnorm folds several branch outputs at once with float32_weight and without a factor")
+            ops.branches_rmsnorm(stream.h, stream.delta, stream.delta_more, self.weight, self.eps, out, row_idx=row_idx, join=stream.delta_join)
+            if row_idx is None:
+                stream.delta = stream.delta_more = stream.delta_join = stream.rounded = None
+            return
         ops.add_rmsnorm(stream.h, stream.delta, self.weight, self.eps, out, row_idx=row_idx,
                         write_residual=row_idx is None, delta_scale=stream.delta_scale)
         if row_idx is None:

@@ -98,7 +98,8 @@ class SpanRotaryPosition(PositionEncoding):
                  scaling: Optional[Mapping[str, float]] = None, unit_rms_eps: Optional[float] = None):
         """``scaling`` (``factor``, ``original``, ``fast``, ``slow``): the frequencies are stretched for contexts longer than
         ``original`` positions, pair by pair (see :meth:`inverse_frequencies`), and cosines and sines are multiplied by
-        ``0.1 ln(factor) + 1``.  ``unit_rms_eps``: after the turn every query and key head is divided by its root mean square
+        ``0.1 ln(factor) + 1``; with ``low`` and ``high`` in place of ``slow`` and ``fast`` the stretch goes by a pair's wavelength
+        and cosines and sines stay as they are.  ``unit_rms_eps``: after the turn every query and key head is divided by its root mean square
         ``sqrt(mean(x^2) + unit_rms_eps)``.  Either option, a cache whose rows are wider than a head or a value size of its
         own takes the kernel ``ops.rotary_norm`` (span at the start of the head); ``dims`` may then be 0 (nothing turns)."""
         plain = scaling is None and unit_rms_eps is None
@@ -115,15 +116,18 @@ class SpanRotaryPosition(PositionEncoding):
         self.unit_rms_eps = float(unit_rms_eps) if unit_rms_eps is not None else None
         self.scaling = None
         self.magnitude = 1.0
+        self.by_wavelength = False
         if scaling is not None:
-            missing = [k for k in ("factor", "original", "fast", "slow") if k not in scaling]
+            self.by_wavelength = "low" in scaling or "high" in scaling
+            keys = ("factor", "original", "low", "high") if self.by_wavelength else ("factor", "original", "fast", "slow")
+            missing = [k for k in keys if k not in scaling]
             if missing:
                 raise ValueError(f"rope_span: scaling lacks {missing}")
-            self.scaling = {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}
-            if not (self.scaling["factor"] > 0.0 and self.scaling["original"] > 0.0 and self.scaling["fast"] > 0.0
-                    and self.scaling["slow"] > 0.0 and self.theta != 1.0):
+            self.scaling = {k: float(scaling[k]) for k in keys}
+            if not (min(self.scaling.values()) > 0.0 and self.theta != 1.0):
                 raise ValueError(f"rope_span: scaling={dict(scaling)} must be positive throughout (and theta differ from 1)")
-            self.magnitude = 0.1 * math.log(self.scaling["factor"]) + 1.0
+            if not self.by_wavelength:
+                self.magnitude = 0.1 * math.log(self.scaling["factor"]) + 1.0
         self._inv_freq: Optional[torch.Tensor] = None
 
     def inverse_frequencies(self) -> torch.Tensor:
@@ -131,10 +135,18 @@ class SpanRotaryPosition(PositionEncoding):
         n)) / (2 ln theta)`` be the pair that makes n full turns over ``original`` positions, ``lo = max(floor(D(fast)), 0)``,
         ``hi = min(ceil(D(slow)), dims - 1)`` and ``m_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)``; the table holds ``f_i
         / factor * m_i + f_i (1 - m_i)``: pairs below ``lo`` keep their frequency, pairs above ``hi`` turn ``factor`` times
-        slower.  Formed in float64 and rounded once."""
+        slower.  By wavelength (``low``, ``high``): with ``l = 2 pi / f``, f stays where ``l < original / high``, becomes ``f / factor``
+        where ``l > original / low``, and between the two ``(1 - s) f / factor + s f`` with ``s = (original / l - low) / (high -
+        low)``.  Formed in float64 and rounded once."""
         i = torch.arange(0, self.dims // 2, dtype=torch.float64)
         f = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / max(self.dims, 1))
-        if self.scaling is not None:
+        if self.by_wavelength:
+            sc = self.scaling
+            turns = sc["original"] * f / (2.0 * math.pi)                        # original / wavelength
+            s = (turns - sc["low"]) / max(sc["high"] - sc["low"], 1e-30)
+            between = (1.0 - s) * f / sc["factor"] + s * f
+            f = torch.where(turns > sc["high"], f, torch.where(turns < sc["low"], f / sc["factor"], between))
+        elif self.scaling is not None:
             sc = self.scaling
 
             def pair_of(turns: float) -> float:
