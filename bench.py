@@ -398,6 +398,27 @@ def sumitar_config(width, heads, ff, window, layers, vocab, experts, top, expert
     return {"architecture": "Sumitar", "vocab": vocab, "width": width, "max_positions": CONTEXT, "norm": {"eps": 1e-5}, "layers": out}
 
 
+def bogivik_config(width, heads, ff, window, layers, vocab, dim=128, **_):
+    """The Bogivik design at the same width, layers, heads, head size, vocabulary and feed-forward as the configurations beside
+    it (all have a gated feed-forward of three matrices): attention over every key with a bias by distance (32 buckets, the
+    farthest from the window's length on), a query temperature and mixed values, and layers of two mixers (attention in
+    chunks of the window's length, half of every head turned with stretched frequencies, beside a matrix memory with heads of
+    64 x 128) by turns."""
+    kv = 2 if heads <= 12 else 4
+    shape = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    scaling = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}
+    out = []
+    for i in range(layers):
+        if i % 2 == 0:
+            layer = {"type": "attention", "mixer": dict(shape, bias_max=window, q_temp={"coef": 0.1, "every": 1024}, v_mix=True)}
+        else:
+            layer = {"type": "parallel", "mixer": {
+                "left": dict(shape, mask={"size": window}, rot={"base": 500000.0, "dims": dim // 2, "scaling": scaling}),
+                "right": {"heads": heads, "dim": dim // 2, "vdim": dim, "gate_cap": 15.0}}}
+        out.append(dict(layer, mlp={"kind": "dense", "ff": (2 * ff // 3 + 7) // 8 * 8}))
+    return {"architecture": "Bogivik", "vocab": vocab, "width": width, "max_positions": CONTEXT, "norm": {"eps": 1e-6}, "layers": out}
+
+
 def measure_design(cfg, vocab, batch, steps, warmup):
     """Prefill of PROMPT_LEN tokens in one step and decode of `batch` requests through the captured greedy step."""
     import torch
@@ -455,6 +476,17 @@ def design_comparison(args):
     rows = []
     for name, size in DESIGN_SIZES.items():
         q = {k: size[k] for k in ("width", "heads", "ff", "window", "layers", "vocab")}
+        if args.designs == "bogivik":
+            # the design beside Kevatar (attention, matrix states, a gated feed-forward) and beside Qwen2
+            qwen = measure_design(qwen2_config_like(**q), size["vocab"], args.batch, steps, warmup)
+            kev = measure_design(kevatar_config(**q), size["vocab"], args.batch, steps, warmup)
+            bog = measure_design(bogivik_config(**q), size["vocab"], args.batch, steps, warmup)
+            rows.append({"size": name, "shape": q, "bogivik": bog, "kevatar": kev, "qwen2_equal_size": qwen,
+                         "prefill_ratio_to_kevatar": round(bog["prefill_tokens_per_s"] / kev["prefill_tokens_per_s"], 3),
+                         "decode_ratio_to_kevatar": round(bog["decode_tokens_per_s"] / kev["decode_tokens_per_s"], 3),
+                         "prefill_ratio": round(bog["prefill_tokens_per_s"] / qwen["prefill_tokens_per_s"], 3),
+                         "decode_ratio": round(bog["decode_tokens_per_s"] / qwen["decode_tokens_per_s"], 3)})
+            continue
         if args.designs == "sumitar":
             # the design beside Kevatar, its closest relative (windowed attention and matrix states), and beside Qwen2
             qwen = measure_design(qwen2_config_like(**q), size["vocab"], args.batch, steps, warmup)
@@ -580,7 +612,7 @@ def main():
     ap.add_argument("--layers", type=int, default=MODEL_1P5B["num_hidden_layers"],
                     help="fewer layers than the model has (same layer sizes), where memory or time needs it")
     ap.add_argument("--no-points", action="store_true", help="skip the batch-1 and batch-64 points")
-    ap.add_argument("--designs", nargs="?", const="baselix", default=None, choices=["baselix", "gibalorn", "kevatar", "sumitar"],
+    ap.add_argument("--designs", nargs="?", const="baselix", default=None, choices=["baselix", "gibalorn", "kevatar", "sumitar", "bogivik"],
                     help="instead of the default workload: prefill and decode of the Baselix design at layer sizes of real "
                          "models (random weights) beside Qwen2 at equal size; '--designs gibalorn' also runs the Gibalorn "
                          "design at those sizes; '--designs kevatar' runs the Kevatar design beside Qwen2 alone; '--designs sumitar' the "

@@ -161,7 +161,7 @@ def chunked_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: di
     v = (h @ w[p + "v"].T + w[p + "v.b"]).view(n, G, dv)
     pos, rot = torch.arange(n), m["rot"]
     q, k = (turn_pairs(z, pos, rot["dims"], rot["base"], rot.get("scaling")) for z in (q, k))
-    chunk = pos // m["mask"]["size"]
+    chunk = pos // (m["mask"]["size"] if m.get("mask") else n)
     seen = (pos[:, None] >= pos[None, :]) & (chunk[:, None] == chunk[None, :])
     o = attend(q, k, v, m["scale"], seen)
     return (o * logistic(h @ w[p + "g"].T)) @ w[p + "o"].T + w[p + "o.b"]

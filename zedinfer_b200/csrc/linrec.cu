@@ -388,6 +388,11 @@ __global__ void __launch_bounds__(COLS * LANES)
 linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec, const float* __restrict__ pv, int tiles) {
     constexpr int DP = LANES * R, NT = COLS * LANES, REC = LrRecord<RULE, DP>::SIZE;
     constexpr int STAGE = LR_WALK_CHUNK * (REC + COLS);                      // a chunk's records, then its values
+    // expgate: fade, write and m of a chunk's tokens, one copy per warp.  A chunk holds as many tokens as a warp has lanes: the
+    // lanes follow the running maximum through the chunk together, then each makes its own token's two exponentials.
+    __shared__ float4 sgates[RULE == LR_EXPGATE ? NT / 32 : 1][RULE == LR_EXPGATE ? LR_WALK_CHUNK : 1];
+    static_assert(LR_WALK_CHUNK == 32, "a lane per token of a chunk");
+    float4* gates = sgates[RULE == LR_EXPGATE ? threadIdx.x >> 5 : 0];
     extern __shared__ __align__(16) float smem[];
     const int seg = blockIdx.x / tiles, tile = blockIdx.x - seg * tiles, h = blockIdx.y;
     const int sub = threadIdx.x % LANES;
@@ -437,6 +442,19 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
         __syncthreads();                                                   // everyone's copies of this chunk have landed
         const float* st = smem + s * STAGE;
         const float* sv = st + LR_WALK_CHUNK * REC + threadIdx.x / LANES;
+        if (RULE == LR_EXPGATE) {
+            const int lane = threadIdx.x & 31;
+            const float gi = lane < cnt ? st[lane * REC + REC - 4] : 0.0f, gf = lane < cnt ? st[lane * REC + REC - 2] : 0.0f;
+            float before = m;
+            for (int t = 0; t < cnt; ++t) {
+                if (t == lane) before = m;
+                m = fmaxf(__shfl_sync(0xffffffffu, gf, t) + m, __shfl_sync(0xffffffffu, gi, t));
+            }
+            float after = before, fade, write;
+            lr_gate_step(after, gi, gf, fade, write);
+            gates[lane] = make_float4(fade, write, after, 0.0f);
+            __syncwarp();
+        }
         int tt = 0;
         // four tokens at a time, in straight-line code
         for (; tt + 4 <= cnt; tt += 4) {
@@ -446,12 +464,11 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
                 const float* r = st + (tt + j) * REC;
                 float kr[R], ks, fade = lam;
                 u[j] = sv[(tt + j) * COLS];
+                mt[j] = 0.0f;
                 if (RULE == LR_EXPGATE) {
-                    float write;
-                    lr_gate_step(m, r[REC - 4], r[REC - 2], fade, write);
-                    u[j] *= write;
+                    const float4 g = gates[tt + j];
+                    fade = g.x; u[j] *= g.y; mt[j] = g.z;
                 }
-                mt[j] = m;
                 lr_token_local<R, LANES, RULE>(S, kr, r + DP, r, r + 2 * DP, fade, sub, ks, qs[j]);
                 qk[j] = r[REC - 3];
                 if (RULE == LR_DELTA) {
@@ -471,14 +488,13 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
         }
         for (; tt < cnt; ++tt) {
             const float* r = st + tt * REC;
-            float fade = lam, vv = sv[tt * COLS];
+            float fade = lam, vv = sv[tt * COLS], mt = 0.0f;
             if (RULE == LR_EXPGATE) {
-                float write;
-                lr_gate_step(m, r[REC - 4], r[REC - 2], fade, write);
-                vv *= write;
+                const float4 g = gates[tt];
+                fade = g.x; vv *= g.y; mt = g.z;
             }
             const float o = lr_walk_token<R, LANES, RULE>(S, r + DP, r, r + 2 * DP, fade, vv, r[REC - 4], r[REC - 3], sub);
-            if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt), h, col, o, m);
+            if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt), h, col, o, mt);
         }
         __syncthreads();                                                   // this chunk's buffer may be filled again
     }
@@ -597,6 +613,20 @@ ZI_EXPORT int zi_linear_state(int rule, const void* q, long long ldq, const void
 // is taken by one warp when there are at least as many groups as warps, else by the whole block, group after group.
 // ---------------------------------------------------------------------------------------
 #define GN_THREADS 256
+__device__ __forceinline__ void load4(const float* p, float* o) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+}
+__device__ __forceinline__ void load4(const bf16* p, float* o) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+}
+__device__ __forceinline__ void store4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(bf16* p, const float* v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
 template <typename T>
 __device__ __forceinline__ float gn_gate(const T* zr, int c, int gate) {
     if (gate == 2) return 1.0f;
@@ -604,7 +634,7 @@ __device__ __forceinline__ float gn_gate(const T* zr, int c, int gate) {
     return gate == 1 ? lr_silu(z) : lr_sigmoid(z);
 }
 
-template <typename T, typename TW>
+template <typename T, typename TW, int V>
 __global__ void __launch_bounds__(GN_THREADS)
 group_rmsnorm_gate_kernel(const float* __restrict__ y, const float* __restrict__ den, const T* __restrict__ z, long long ldz, const TW* __restrict__ w, int w_len,
                           T* __restrict__ out, int inner, int n_groups, float eps, int gate) {
@@ -614,6 +644,45 @@ group_rmsnorm_gate_kernel(const float* __restrict__ y, const float* __restrict__
     const T* zr = gate == 2 ? nullptr : z + (size_t)n * ldz;
     T* orow = out + (size_t)n * inner;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if constexpr (V > 0) {
+        // a warp per group, four entries per access and V such accesses per lane, everything asked for before the sum is taken
+        for (int g = warp; g < n_groups; g += GN_THREADS / 32) {
+            const float dv = den ? 1.0f / den[(size_t)n * n_groups + g] : 1.0f;
+            float yv[V][4], wv[V][4], zv[V][4], ss = 0.0f;
+#pragma unroll
+            for (int k = 0; k < V; ++k) {
+                const int j = (k * 32 + lane) * 4;
+                if (j < gw) {
+                    const int c = g * gw + j;
+                    load4(yr + c, yv[k]);
+                    load4(w + c % w_len, wv[k]);
+                    if (gate != 2) load4(zr + c, zv[k]);
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < V; ++k)
+                if ((k * 32 + lane) * 4 < gw) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) { yv[k][e] *= dv; ss = fmaf(yv[k][e], yv[k][e], ss); }
+                }
+            ss = warp_sum(ss);
+            const float r = 1.0f / sqrtf(ss / (float)gw + eps);
+#pragma unroll
+            for (int k = 0; k < V; ++k) {
+                const int j = (k * 32 + lane) * 4;
+                if (j < gw) {
+                    float o[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float gt = gate == 2 ? 1.0f : (gate == 1 ? lr_silu(zv[k][e]) : lr_sigmoid(zv[k][e]));
+                        o[e] = yv[k][e] * r * wv[k][e] * gt;
+                    }
+                    store4(orow + g * gw + j, o);
+                }
+            }
+        }
+        return;
+    }
     if (n_groups >= GN_THREADS / 32) {
         for (int g = warp; g < n_groups; g += GN_THREADS / 32) {
             const float dv = den ? 1.0f / den[(size_t)n * n_groups + g] : 1.0f;
@@ -647,9 +716,13 @@ ZI_EXPORT int zi_group_rmsnorm_gate(const float* y, const float* den, const void
     if (inner <= 0 || n_groups <= 0 || inner % n_groups) return zi_fail("group_rmsnorm_gate: %d groups do not divide %d", n_groups, inner);
     if (gate < 0 || gate > 2 || (gate != 2 && !z)) return zi_fail("group_rmsnorm_gate: gate %d is none of 0 (sigmoid), 1 (SiLU), 2 (none), or its input is missing", gate);
     if (w_len <= 0 || inner % w_len) return zi_fail("group_rmsnorm_gate: a weight of %d entries does not tile a row of %d", w_len, inner);
+    // which form runs depends on the sizes and on where the buffers start, never on the rows of the step
+    const int gw = inner / n_groups;
+    const bool vec = gw % 4 == 0 && gw <= 512 && w_len % 4 == 0 && (!z || ldz % 4 == 0) && (((size_t)y | (size_t)z | (size_t)w | (size_t)out) & 15) == 0;
     ZI_DISPATCH(dtype, T, ZI_DISPATCH(w_dtype, TW, {
-        group_rmsnorm_gate_kernel<T, TW><<<n_tokens, GN_THREADS, 0, stream>>>(y, den, (const T*)z, ldz, (const TW*)w, w_len, (T*)out, inner,
-                                                                            n_groups, eps, gate);
+        auto kernel = !vec ? group_rmsnorm_gate_kernel<T, TW, 0> : gw <= 128 ? group_rmsnorm_gate_kernel<T, TW, 1>
+                           : gw <= 256 ? group_rmsnorm_gate_kernel<T, TW, 2> : group_rmsnorm_gate_kernel<T, TW, 4>;
+        kernel<<<n_tokens, GN_THREADS, 0, stream>>>(y, den, (const T*)z, ldz, (const TW*)w, w_len, (T*)out, inner, n_groups, eps, gate);
     }););
     return zi_check_launch("group_rmsnorm_gate");
 }

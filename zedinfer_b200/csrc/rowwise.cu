@@ -1330,7 +1330,7 @@ branches_rmsnorm_kernel(const FoldArgs a, T* __restrict__ out) {
         float s1 = 0.0f, s2 = 0.0f, unused = 0.0f;
 #pragma unroll
         for (int c = 0; c < C; ++c) {
-            const int j = (c * 256 + threadIdx.x) * 8;
+            const int j = (c * (int)blockDim.x + (int)threadIdx.x) * 8;
             if (j < hidden) {
                 load8(a.h + base + j, v[c]);
                 if (a.w) load8(a.w + j, w[c]);
@@ -1367,7 +1367,7 @@ branches_rmsnorm_kernel(const FoldArgs a, T* __restrict__ out) {
         float ss = 0.0f;
 #pragma unroll
         for (int c = 0; c < C; ++c) {
-            const int j = (c * 256 + threadIdx.x) * 8;
+            const int j = (c * (int)blockDim.x + (int)threadIdx.x) * 8;
             if (j < hidden) {
                 if (a.y) {
 #pragma unroll
@@ -1385,7 +1385,7 @@ branches_rmsnorm_kernel(const FoldArgs a, T* __restrict__ out) {
         const float rr = 1.0f / sqrtf(ss * inv_n + a.eps);
 #pragma unroll
         for (int c = 0; c < C; ++c) {
-            const int j = (c * 256 + threadIdx.x) * 8;
+            const int j = (c * (int)blockDim.x + (int)threadIdx.x) * 8;
             if (j < hidden) {
 #pragma unroll
                 for (int e = 0; e < 8; ++e) v[c][e] = v[c][e] * rr * w[c][e];
@@ -1442,9 +1442,10 @@ ZI_EXPORT int zi_branches_rmsnorm(float* h, const void* y, int y_parts, const vo
     const bool vec = hidden % 8 == 0 && hidden <= 8192 && part_stride % 8 == 0 &&
                      (((size_t)h | (size_t)y | (size_t)y2 | (size_t)f | (size_t)out | (size_t)w1 | (size_t)w2 | (size_t)w) & 15) == 0;
     ZI_DISPATCH(dtype, T, {
-        if (vec && hidden <= 2048) branches_rmsnorm_kernel<T, 1><<<rows, 256, 0, stream>>>(a, (T*)out);
-        else if (vec && hidden <= 4096) branches_rmsnorm_kernel<T, 2><<<rows, 256, 0, stream>>>(a, (T*)out);
-        else if (vec) branches_rmsnorm_kernel<T, 4><<<rows, 256, 0, stream>>>(a, (T*)out);
+        const int c = hidden <= 2048 ? 1 : (hidden <= 4096 ? 2 : 4), threads = (hidden / 8 + c * 32 - 1) / (c * 32) * 32;   // no idle warps
+        if (vec && c == 1) branches_rmsnorm_kernel<T, 1><<<rows, threads, 0, stream>>>(a, (T*)out);
+        else if (vec && c == 2) branches_rmsnorm_kernel<T, 2><<<rows, threads, 0, stream>>>(a, (T*)out);
+        else if (vec) branches_rmsnorm_kernel<T, 4><<<rows, threads, 0, stream>>>(a, (T*)out);
         else {
             const size_t smem = (size_t)hidden * sizeof(float);
             if (smem > 48 * 1024) return zi_fail("branches_rmsnorm: hidden=%d is not supported", hidden);
