@@ -227,11 +227,11 @@ __device__ __forceinline__ float lr_walk_token(float (&S)[R], const float* sk, c
     return fmaf(qk, u, qs);
 }
 
-// A column's output of one token: the read-out, or (expgate, column vdim) the divisor of the head's read-outs.
+// A column's output of one token: the read-out o, or (expgate, the key sum's column) the divisor of the head's read-outs, at
+// least exp(-m).
 template <int RULE>
-__device__ __forceinline__ void lr_emit(const LinearStateArgs& p, size_t n, int h, int col, float o, float m) {
-    if (col < p.vdim) p.y[n * ((size_t)p.heads * p.vdim) + (size_t)h * p.vdim + col] = o;
-    else if (RULE == LR_EXPGATE && col == p.vdim) p.den[n * p.heads + h] = fmaxf(fabsf(o), expf(-m)) + LR_DEN_EPS;
+__device__ __forceinline__ float lr_column_out(float o, float least, bool is_den) {
+    return RULE == LR_EXPGATE && is_den ? fmaxf(fabsf(o), least) + LR_DEN_EPS : o;
 }
 
 // ---- the walk that makes its own inputs ready (steps of single tokens) -----------------------------------------------------
@@ -273,6 +273,10 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
     const float rate = RULE == LR_DELTA ? expf(p.a_log[h]) : 0.0f;
     float* smax = RULE == LR_EXPGATE && srow ? p.state + (size_t)slot * p.slot_stride + (size_t)p.heads * columns * dim + (size_t)h * columns + col : nullptr;
     float m = smax ? *smax : 0.0f;
+    // where a column's outputs go: the read-outs, or (expgate, the last column) the heads' divisors
+    const bool is_den = RULE == LR_EXPGATE && col == p.vdim, writes = sub == 0 && live;
+    const size_t ld = is_den ? (size_t)p.heads : (size_t)p.heads * p.vdim;
+    float* dst = is_den ? p.den + h : p.y + (size_t)h * p.vdim + col;
 
     for (int c0 = t0; c0 < t1; c0 += LR_CHUNK) {
         const int cnt = min(LR_CHUNK, t1 - c0);
@@ -308,7 +312,7 @@ linear_state_kernel(const LinearStateArgs p, int tiles) {
                 vv *= write;
             }
             const float o = lr_walk_token<R, LANES, RULE>(S, sk + tt * DP, sq + tt * DP, sg + tt * DP, fade, vv, sbeta[tt], sqk[tt], sub);
-            if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt), h, col, o, m);
+            if (writes) dst[(size_t)(c0 + tt) * ld] = lr_column_out<RULE>(o, RULE == LR_EXPGATE ? expf(-m) : 0.0f, is_den);
         }
     }
     if (smax && sub == 0) *smax = m;
@@ -388,7 +392,7 @@ __global__ void __launch_bounds__(COLS * LANES)
 linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec, const float* __restrict__ pv, int tiles) {
     constexpr int DP = LANES * R, NT = COLS * LANES, REC = LrRecord<RULE, DP>::SIZE;
     constexpr int STAGE = LR_WALK_CHUNK * (REC + COLS);                      // a chunk's records, then its values
-    // expgate: fade, write and m of a chunk's tokens, one copy per warp.  A chunk holds as many tokens as a warp has lanes: the
+    // expgate: fade, write and exp(-m) of a chunk's tokens, one copy per warp.  A chunk holds as many tokens as a warp has lanes: the
     // lanes follow the running maximum through the chunk together, then each makes its own token's two exponentials.
     __shared__ float4 sgates[RULE == LR_EXPGATE ? NT / 32 : 1][RULE == LR_EXPGATE ? LR_WALK_CHUNK : 1];
     static_assert(LR_WALK_CHUNK == 32, "a lane per token of a chunk");
@@ -415,6 +419,10 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
     const float lam = RULE == LR_DECAY ? p.decay[h] : 0.0f;
     float* smax = RULE == LR_EXPGATE && srow ? p.state + (size_t)slot * p.slot_stride + (size_t)p.heads * columns * dim + (size_t)h * columns + col : nullptr;
     float m = smax ? *smax : 0.0f;
+    // where a column's outputs go: the read-outs, or (expgate, the last column) the heads' divisors
+    const bool is_den = RULE == LR_EXPGATE && col == p.vdim, writes = sub == 0 && live;
+    const size_t ld = is_den ? (size_t)p.heads : (size_t)p.heads * p.vdim;
+    float* dst = is_den ? p.den + h : p.y + (size_t)h * p.vdim + col;
 
     auto fetch = [&](int c0, float* dst) {
         const int cnt = min(LR_WALK_CHUNK, t1 - c0);
@@ -444,30 +452,32 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
         const float* sv = st + LR_WALK_CHUNK * REC + threadIdx.x / LANES;
         if (RULE == LR_EXPGATE) {
             const int lane = threadIdx.x & 31;
-            const float gi = lane < cnt ? st[lane * REC + REC - 4] : 0.0f, gf = lane < cnt ? st[lane * REC + REC - 2] : 0.0f;
+            // lanes past the chunk's tokens leave the maximum as it is
+            const float gi = lane < cnt ? st[lane * REC + REC - 4] : -INFINITY, gf = lane < cnt ? st[lane * REC + REC - 2] : 0.0f;
             float before = m;
-            for (int t = 0; t < cnt; ++t) {
-                if (t == lane) before = m;
+#pragma unroll
+            for (int t = 0; t < LR_WALK_CHUNK; ++t) {
+                before = t == lane ? m : before;
                 m = fmaxf(__shfl_sync(0xffffffffu, gf, t) + m, __shfl_sync(0xffffffffu, gi, t));
             }
             float after = before, fade, write;
             lr_gate_step(after, gi, gf, fade, write);
-            gates[lane] = make_float4(fade, write, after, 0.0f);
+            gates[lane] = make_float4(fade, write, expf(-after), 0.0f);
             __syncwarp();
         }
         int tt = 0;
         // four tokens at a time, in straight-line code
         for (; tt + 4 <= cnt; tt += 4) {
-            float qs[4], u[4], qk[4], mt[4];
+            float qs[4], u[4], qk[4], least[4];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float* r = st + (tt + j) * REC;
                 float kr[R], ks, fade = lam;
                 u[j] = sv[(tt + j) * COLS];
-                mt[j] = 0.0f;
+                least[j] = 0.0f;
                 if (RULE == LR_EXPGATE) {
                     const float4 g = gates[tt + j];
-                    fade = g.x; u[j] *= g.y; mt[j] = g.z;
+                    fade = g.x; u[j] *= g.y; least[j] = g.z;
                 }
                 lr_token_local<R, LANES, RULE>(S, kr, r + DP, r, r + 2 * DP, fade, sub, ks, qs[j]);
                 qk[j] = r[REC - 3];
@@ -484,17 +494,17 @@ linear_state_walk_kernel(const LinearStateArgs p, const float* __restrict__ rec,
                 for (int j = 0; j < 4; ++j) qs[j] += __shfl_xor_sync(0xffffffffu, qs[j], o);
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-                if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt + j), h, col, fmaf(qk[j], u[j], qs[j]), mt[j]);
+                if (writes) dst[(size_t)(c0 + tt + j) * ld] = lr_column_out<RULE>(fmaf(qk[j], u[j], qs[j]), least[j], is_den);
         }
         for (; tt < cnt; ++tt) {
             const float* r = st + tt * REC;
-            float fade = lam, vv = sv[tt * COLS], mt = 0.0f;
+            float fade = lam, vv = sv[tt * COLS], least = 0.0f;
             if (RULE == LR_EXPGATE) {
                 const float4 g = gates[tt];
-                fade = g.x; vv *= g.y; mt = g.z;
+                fade = g.x; vv *= g.y; least = g.z;
             }
             const float o = lr_walk_token<R, LANES, RULE>(S, r + DP, r, r + 2 * DP, fade, vv, r[REC - 4], r[REC - 3], sub);
-            if (sub == 0) lr_emit<RULE>(p, (size_t)(c0 + tt), h, col, o, mt);
+            if (writes) dst[(size_t)(c0 + tt) * ld] = lr_column_out<RULE>(o, least, is_den);
         }
         __syncthreads();                                                   // this chunk's buffer may be filled again
     }

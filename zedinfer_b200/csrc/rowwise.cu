@@ -1146,11 +1146,29 @@ qk_norm_append_kernel(const T* __restrict__ x, T* __restrict__ q_out, T* __restr
     float* row = qp_smem;
     float* cs = row + (qk_len + 3) / 4 * 4;
     float* factor = cs + a.rot_dims;
+    // the row and the position are asked for together; the page number, which waits for the position, is asked for behind them
     const int p = pos[n];
     const int seg = tok_seg ? tok_seg[n] : n;
+    const T* xr = x + (size_t)n * a.ldx;
+    float sq = 0.0f, sk = 0.0f, unused = 0.0f;
+    if (VEC) {
+        for (int j = threadIdx.x * 8; j < qk_len; j += QP_THREADS * 8) {
+            float v[8], s = 0.0f;
+            load8(xr + j, v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+            store8(row + j, v);
+            if (j < q_len) sq += s; else sk += s;      // a group of eight lies in one head
+        }
+    } else {
+        for (int j = threadIdx.x; j < qk_len; j += QP_THREADS) {
+            const float v = to_f32<T>(xr[j]);
+            row[j] = v;
+            if (j < q_len) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
+        }
+    }
     const int page = tables[(size_t)seg * a.max_blocks + p / a.page_size];
     T* page_base = cache + (size_t)page * a.page_stride + (size_t)(p % a.page_size) * a.row_dim;
-    const T* xr = x + (size_t)n * a.ldx;
     // values need nothing of the rest
     const T* vr = xr + qk_len;
     const T* fr = v_first ? v_first + (size_t)n * a.ld_first : nullptr;
@@ -1188,23 +1206,6 @@ qk_norm_append_kernel(const T* __restrict__ x, T* __restrict__ q_out, T* __restr
         cs[half + i] = s * a.mag;
     }
     const float heat = a.heat_every > 0.0f ? fmaf(a.heat_coef, logf(floorf((float)(p + 1) / a.heat_every) + 1.0f), 1.0f) : 1.0f;
-    float sq = 0.0f, sk = 0.0f, unused = 0.0f;
-    if (VEC) {
-        for (int j = threadIdx.x * 8; j < qk_len; j += QP_THREADS * 8) {
-            float v[8], s = 0.0f;
-            load8(xr + j, v);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
-            store8(row + j, v);
-            if (j < q_len) sq += s; else sk += s;      // a group of eight lies in one head
-        }
-    } else {
-        for (int j = threadIdx.x; j < qk_len; j += QP_THREADS) {
-            const float v = to_f32<T>(xr[j]);
-            row[j] = v;
-            if (j < q_len) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
-        }
-    }
     if (a.norm == 2) {
         block_sum3(sq, sk, unused, scratch);
         const float rq = 1.0f / sqrtf(sq / (float)q_len + a.eps), rk = 1.0f / sqrtf(sk / (float)(qk_len - q_len) + a.eps);
@@ -1230,20 +1231,43 @@ qk_norm_append_kernel(const T* __restrict__ x, T* __restrict__ q_out, T* __restr
         const float r = factor[h], last = h < a.n_q ? heat : 1.0f;
         auto normed = [&](int d) { return w ? hr[d] * r * w[d] : hr[d]; };
         float o[8];
+        if (VEC && d0 + 8 <= a.qk_dim && (d0 >= a.rot_dims || (a.interleaved && a.rot_dims % 8 == 0))) {
+            // the eight entries, their weights and (four whole pairs) their angles as vectors
+            float v[8];
+            load8(hr + d0, v);
+            if (w) {
+                float wv[8];
+                load8(w + d0, wv);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-            const int d = d0 + e;
-            float v = 0.0f;
-            if (d < a.rot_dims) {
-                const int i = a.interleaved ? d >> 1 : (d < half ? d : d - half);
-                const int lo_at = a.interleaved ? d & ~1 : i, hi_at = a.interleaved ? d | 1 : i + half;
-                float olo, ohi;
-                rotate_pair(normed(lo_at), normed(hi_at), cs[i], cs[half + i], &olo, &ohi);
-                v = d == lo_at ? olo : ohi;
-            } else if (d < a.qk_dim) {
-                v = normed(d);
+                for (int e = 0; e < 8; ++e) v[e] = v[e] * r * wv[e];
             }
-            o[e] = v * last;
+            if (d0 < a.rot_dims) {
+                const float4 c4 = *reinterpret_cast<const float4*>(cs + d0 / 2), s4 = *reinterpret_cast<const float4*>(cs + half + d0 / 2);
+                const float c[4] = {c4.x, c4.y, c4.z, c4.w}, sn[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float lo = v[2 * i], hi = v[2 * i + 1];
+                    rotate_pair(lo, hi, c[i], sn[i], &v[2 * i], &v[2 * i + 1]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = v[e] * last;
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int d = d0 + e;
+                float v = 0.0f;
+                if (d < a.rot_dims) {
+                    const int i = a.interleaved ? d >> 1 : (d < half ? d : d - half);
+                    const int lo_at = a.interleaved ? d & ~1 : i, hi_at = a.interleaved ? d | 1 : i + half;
+                    float olo, ohi;
+                    rotate_pair(normed(lo_at), normed(hi_at), cs[i], cs[half + i], &olo, &ohi);
+                    v = d == lo_at ? olo : ohi;
+                } else if (d < a.qk_dim) {
+                    v = normed(d);
+                }
+                o[e] = v * last;
+            }
         }
         T* dst = h < a.n_q ? q_out + ((size_t)n * a.n_q + h) * a.row_dim : page_base + (size_t)(h - a.n_q) * a.page_size * a.row_dim;
         store8(dst + d0, o);
@@ -1264,7 +1288,7 @@ ZI_EXPORT int zi_qk_norm_append(const void* x, int dtype, long long ldx, void* q
     if (rot_dims > 0 && !inv_freq) return zi_fail("qk_norm_append: a turned span needs its frequencies");
     const size_t align = dtype == ZI_BF16 ? 15 : 31;
     if ((((uintptr_t)q_out | (uintptr_t)cache) & align) || page_stride % 8 || kv_stride % 8) return zi_fail("qk_norm_append: q_out and cache must be aligned for eight entries");
-    const bool vec = qk_dim % 8 == 0 && v_dim % 8 == 0 && ldx % 8 == 0 && ((uintptr_t)x & align) == 0 &&
+    const bool vec = qk_dim % 8 == 0 && v_dim % 8 == 0 && ldx % 8 == 0 && ((uintptr_t)x & align) == 0 && (((uintptr_t)qw | (uintptr_t)kw) & 15) == 0 &&
                      (!v_first || (ld_first % 8 == 0 && ((uintptr_t)v_first & align) == 0));
     const size_t smem = ((size_t)((n_q + n_k) * qk_dim + 3) / 4 * 4 + rot_dims + n_q + n_k) * sizeof(float);
     if (smem > 200 * 1024) return zi_fail("qk_norm_append: %d + %d heads of %d entries are too many for one block", n_q, n_k, qk_dim);
