@@ -616,7 +616,7 @@ def main():
                     help="instead of the default workload: prefill and decode of the Baselix design at layer sizes of real "
                          "models (random weights) beside Qwen2 at equal size; '--designs gibalorn' also runs the Gibalorn "
                          "design at those sizes; '--designs kevatar' runs the Kevatar design beside Qwen2 alone; '--designs sumitar' the "
-                         "Sumitar design beside Kevatar and Qwen2")
+                         "Sumitar design beside Kevatar and Qwen2, '--designs bogivik' the Bogivik design beside the same two")
     args = ap.parse_args()
 
     if args.impl == "reference":

@@ -325,7 +325,7 @@ def test_one_key_answers_just_inside_a_chunk_and_none_just_outside(dtype, dim, v
 
 
 @pytest.mark.parametrize("dtype", BOTH)
-@pytest.mark.parametrize("dim,vdim,rows,farthest,page", [(32, 24, 16, 240, 16), (64, 64, 32, 700, 16), (128, 128, 10, 130, 16), (64, 64, 6, 90, 24), (16, 8, 12, 2000, 4)])
+@pytest.mark.parametrize("dim,vdim,rows,farthest,page", [(32, 24, 14, 250, 16), (64, 64, 32, 700, 16), (128, 128, 10, 130, 16), (64, 64, 6, 90, 24), (16, 8, 12, 2000, 4)])
 @pytest.mark.parametrize("bucket", ["zero", "half", "inner", "last"])
 def test_a_bucket_that_stands_out_answers_from_its_first_distance_to_its_last(dtype, dim, vdim, rows, farthest, page, bucket):
     """Scores all zero but for one bucket's large number: a query gets the mean of exactly the values whose distance lies in that

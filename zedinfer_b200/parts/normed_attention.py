@@ -18,8 +18,8 @@ With ``H`` query heads and ``G`` key/value heads (query head h reads key/value h
     ``gate``             the concatenated heads are multiplied entry by entry by sigmoid(Wg x)
     out = Wo heads       (+ a bias with ``out_bias``)
 
-``bucket(n)`` with B = ``bias_rows`` rows and D = ``bias_max``: n below B/2, else ``min(B - 1, B/2 + floor(ln(n / (B/2)) / ln(D /
-(B/2)) (B - B/2)))``: from D on every distance shares the last row.  The table is laid out by distance once, when it is
+``bucket(n)`` with R = ``bias_rows`` rows, half of them (h = R // 2) for single distances: n itself below h; from there on
+``h + floor((R - h) log_b(n / h))`` with ``b = bias_max / h``, never beyond R - 1: from ``bias_max`` on every distance shares the last row.  The table is laid out by distance once, when it is
 bound, so that the attention kernels look a distance up.
 
 Norms, turn, temperature and mixing happen in one kernel on the float32 value of each projected entry, and what attention

@@ -135,9 +135,9 @@ class SpanRotaryPosition(PositionEncoding):
         n)) / (2 ln theta)`` be the pair that makes n full turns over ``original`` positions, ``lo = max(floor(D(fast)), 0)``,
         ``hi = min(ceil(D(slow)), dims - 1)`` and ``m_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)``; the table holds ``f_i
         / factor * m_i + f_i (1 - m_i)``: pairs below ``lo`` keep their frequency, pairs above ``hi`` turn ``factor`` times
-        slower.  By wavelength (``low``, ``high``): with ``l = 2 pi / f``, f stays where ``l < original / high``, becomes ``f / factor``
-        where ``l > original / low``, and between the two ``(1 - s) f / factor + s f`` with ``s = (original / l - low) / (high -
-        low)``.  Formed in float64 and rounded once."""
+        slower.  By wavelength (``low``, ``high``): a pair that makes more than ``high`` turns over ``original`` positions (``n =
+        original f / (2 pi)``) keeps its frequency, one that makes fewer than ``low`` turns ``factor`` times slower, and between
+        the two the result moves from one to the other with n, linearly.  Formed in float64 and rounded once."""
         i = torch.arange(0, self.dims // 2, dtype=torch.float64)
         f = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / max(self.dims, 1))
         if self.by_wavelength:
