@@ -506,7 +506,7 @@ decode_attention_merge_kernel(const float* __restrict__ part, bf16* __restrict__
     out[((size_t)n * n_heads + h) * HD + d] = __float2bfloat16_rn(acc / L);
 }
 
-template <int HD, int DT_KEYS, int CL>
+template <int HD, int DT_KEYS, int CL, bool BIAS>      // BIAS false: `bias` is not looked at
 __global__ void __launch_bounds__(ATT_THREADS)
 decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* __restrict__ q, bf16* __restrict__ out,
                             const int* __restrict__ tables, const int* __restrict__ tok_seg, const int* __restrict__ pos,
@@ -650,7 +650,7 @@ decode_attention_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const bf
         float S[DT_KEYS / 8][4];
         qk_scores_tma<HD, DT_KEYS / 8>(S, qf, sK, lane);
         cap_scores<DT_KEYS / 8>(S, cap_in);
-        if (bias.table) bias_scores<DT_KEYS / 8>(S, bias0, bias1, P - key0, P - key0, bias.len - 1, bias_inv, lane);
+        if (BIAS) bias_scores<DT_KEYS / 8>(S, bias0, bias1, P - key0, P - key0, bias.len - 1, bias_inv, lane);
         if (key0 >= lo && key0 + DT_KEYS - 1 <= P) softmax_step<HD, DT_KEYS / 8, false>(S, O, m, l, key0, lane, lo, P, lo, P, scale2);
         else softmax_step<HD, DT_KEYS / 8, true>(S, O, m, l, key0, lane, lo, P, lo, P, scale2);
         pv_accumulate_tma<HD, DT_KEYS / 8>(O, S, sV, lane);
@@ -958,9 +958,9 @@ static int dt_max_clusters() {
     attr[0].val.clusterDim.x = DEC_CLUSTER; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
     cfg.attrs = attr; cfg.numAttrs = 1;
     cfg.gridDim = dim3(DEC_CLUSTER, 64, 1); cfg.blockDim = dim3(ATT_THREADS); cfg.dynamicSmemBytes = dt_smem<HD, KEYS>();
-    if (set_smem(decode_attention_tma_kernel<HD, KEYS, DEC_CLUSTER>, cfg.dynamicSmemBytes, "decode_attention_tma")) return -1;
+    if (set_smem(decode_attention_tma_kernel<HD, KEYS, DEC_CLUSTER, false>, cfg.dynamicSmemBytes, "decode_attention_tma")) return -1;
     int n = 0;
-    if (cudaOccupancyMaxActiveClusters(&n, decode_attention_tma_kernel<HD, KEYS, DEC_CLUSTER>, &cfg) != cudaSuccess) { cudaGetLastError(); return -1; }
+    if (cudaOccupancyMaxActiveClusters(&n, decode_attention_tma_kernel<HD, KEYS, DEC_CLUSTER, false>, &cfg) != cudaSuccess) { cudaGetLastError(); return -1; }
     cached = n > 0 ? n : -1;
     return cached;
 }
@@ -972,9 +972,9 @@ struct DtArgs {
     DistanceBias bias; float bias_inv;
 };
 
-template <int HD, int KEYS, int CL>
-static cudaError_t dt_launch(const DtArgs& a) {
-    if (set_smem(decode_attention_tma_kernel<HD, KEYS, CL>, dt_smem<HD, KEYS>(), "decode_attention_tma")) return cudaErrorInvalidValue;
+template <int HD, int KEYS, int CL, bool BIAS>
+static cudaError_t dt_launch_form(const DtArgs& a) {
+    if (set_smem(decode_attention_tma_kernel<HD, KEYS, CL, BIAS>, dt_smem<HD, KEYS>(), "decode_attention_tma")) return cudaErrorInvalidValue;
     cudaLaunchConfig_t cfg;
     memset(&cfg, 0, sizeof(cfg));
     cudaLaunchAttribute attr[2];
@@ -989,11 +989,13 @@ static cudaError_t dt_launch(const DtArgs& a) {
     cfg.attrs = attr; cfg.numAttrs = blocks <= 200 ? 2 : 1;
     cfg.gridDim = dim3(CL, a.n_kv_heads * a.q_blocks * a.n_splits, a.n_tokens); cfg.blockDim = dim3(ATT_THREADS);
     cfg.dynamicSmemBytes = dt_smem<HD, KEYS>(); cfg.stream = a.stream;
-    return cudaLaunchKernelEx(&cfg, decode_attention_tma_kernel<HD, KEYS, CL>, *a.mkv, (const bf16*)a.q, (bf16*)a.out, a.tables,
+    return cudaLaunchKernelEx(&cfg, decode_attention_tma_kernel<HD, KEYS, CL, BIAS>, *a.mkv, (const bf16*)a.q, (bf16*)a.out, a.tables,
                               a.tok_seg, a.pos, a.status, a.n_heads, a.n_kv_heads, a.q_blocks, a.page_size, a.box_rows,
                               a.max_blocks, a.window, a.scale2, a.n_splits, a.min_split_tiles, a.part, a.kv_box, a.sinks, a.one_plane,
                               a.cap_in, a.bias, a.bias_inv);
 }
+template <int HD, int KEYS, int CL>
+static cudaError_t dt_launch(const DtArgs& a) { return a.bias.table ? dt_launch_form<HD, KEYS, CL, true>(a) : dt_launch_form<HD, KEYS, CL, false>(a); }
 template <int HD>
 static cudaError_t dt_dispatch(const DtArgs& a, int keys, int cl) {
     if (keys == 32) return dt_launch<HD, 32, DEC_CLUSTER>(a);
